@@ -30,12 +30,21 @@ class RMSGainsSpec:
     """One RMS statistic, several gains: y_k = x / sqrt(mean(x^2) + eps) * gain_k for every name in ``names`` (the
     gains' local tensor names; an empty name is the norm's prefix alone).  The sublayers of a layer that all read
     the same residual through norms of their own get their inputs from one pass over it.  ``one_plus``: the tensors
-    hold the gains minus one: the gain is 1 + tensor."""
+    hold the gains minus one: the gain is 1 + tensor.  ``scalar``: the tensors hold one number, the gain of every element."""
     size: int
     eps: float
     names: Tuple[str, ...] = ("",)
     kind: str = "rms_gains"
     one_plus: bool = False
+    scalar: bool = False
+
+
+@dataclass(frozen=True)
+class NoNormSpec:
+    """No norm in front of a sublayer: it reads the residual itself (after whatever is pending has joined it), in the
+    compute dtype."""
+    size: int
+    kind: str = "no_norm"
 
 
 @dataclass(frozen=True)
@@ -119,6 +128,14 @@ class AttentionSpec:
     ``qk_norm_span``: "head" (the norm runs over each head's elements, one gain of the head's size for all heads) or
     "all" (over the whole q projection, and the whole k projection, of a token at once, gains of those sizes);
     ``qk_norm_names``: the two gains' local tensor names.
+
+    ``unit_values``: each head's value is divided by its root mean square (eps ``unit_eps``, no gain) and cached so.
+    ``temperature`` (None or (coef, every)): the query at position p is multiplied by
+    1 + coef ln(floor((p + 1) / every) + 1), after its norms.  ``bias_rows`` > 0: a learned bias on the score by distance
+    (tensor ``bias_name`` [bias_rows, num_heads]), added after the scale and the soft cap: with h = bias_rows // 2 row n
+    serves distance n < h, and row h + floor(ln(n / h) / ln(bias_far / h) (bias_rows - h)), at most the last one, the
+    distances from h on.  ``own_kv`` False: the layer has no projections of keys and values and reads the cache entry
+    that another layer of the same head counts and sizes writes.
     """
     hidden_size: int
     num_heads: int
@@ -143,6 +160,12 @@ class AttentionSpec:
     gate_name: str = "g"
     qk_norm_span: str = "head"
     qk_norm_names: Tuple[str, str] = ("q_norm.weight", "k_norm.weight")
+    unit_values: bool = False
+    temperature: Optional[Tuple[float, float]] = None
+    bias_rows: int = 0
+    bias_far: float = 0.0
+    bias_name: str = "rel"
+    own_kv: bool = True
 
 
 @dataclass(frozen=True)
@@ -192,7 +215,10 @@ class GatedDeltaSpec:
     ``num_qk_heads`` query/key heads; q, k and v pass a causal convolution of ``conv`` taps per channel and silu, q and
     k are made unit vectors; the decay comes from a low-rank projection (inner size ``decay_rank``), a bias and a rate
     per head; the heads' outputs are RMS-normed over ``vdim`` (one gain for all heads, ``eps``) and gated with the
-    sigmoid of another low-rank projection (``gate_rank``)."""
+    sigmoid of another low-rank projection (``gate_rank``).
+
+    ``decay`` "head": one decay per head instead of one per key channel, from a projection of ``num_heads`` rows
+    (tensor "a").  ``gate`` "full": the gate is one projection (tensor "g"), not a low-rank one; ``gate_fn``: "sigmoid" or "silu"."""
     hidden_size: int
     num_heads: int
     num_qk_heads: int
@@ -203,6 +229,9 @@ class GatedDeltaSpec:
     gate_rank: int
     eps: float
     kind: str = "gated_delta"
+    decay: str = "channel"
+    gate: str = "low_rank"
+    gate_fn: str = "sigmoid"
 
 
 @dataclass(frozen=True)
@@ -255,7 +284,10 @@ class MoESpec:
     ``score`` "sigmoid": a score is the sigmoid of its router output alone.  ``groups`` > 1: the router's outputs form
     that many equal groups of neighbours; a group's score is the sum of its ``group_top`` largest choice scores (score
     plus correction), and only experts of the ``group_keep`` best groups can be chosen.  ``renormalize`` False: the
-    weights are the chosen scores as they are; ``route_scale`` multiplies them."""
+    weights are the chosen scores as they are; ``route_scale`` multiplies them.
+
+    ``route`` "table": no router; an integer table (tensor ``table_name`` [table_rows, top]) gives every token id its
+    experts, each with weight 1 / top."""
     hidden_size: int
     experts: int
     top: int
@@ -269,6 +301,19 @@ class MoESpec:
     group_top: int = 2
     renormalize: bool = True
     route_scale: float = 1.0
+    route: str = "scores"
+    table_rows: int = 0
+    table_name: str = "table"
+
+
+@dataclass(frozen=True)
+class TokenSideSpec:
+    """A sublayer fed by the token itself: proj(gelu_tanh(gate x) * e), e the columns [start, start + size) of the
+    token's row in a table that all layers share (the embedding's ``side_name`` table).  No biases."""
+    hidden_size: int
+    size: int
+    start: int
+    kind: str = "token_side"
 
 
 @dataclass(frozen=True)
@@ -298,13 +343,14 @@ class PostNormSpec:
     x <- x + scale * (y / sqrt(mean(y^2) + eps) * gain), y the sublayer's output (a weighted sum of several outputs is
     taken first).  ``gain_name``: the gain's tensor; ``one_plus``: it holds the gain minus one (gain = 1 + tensor);
     ``scale_name``: a vector of the residual's size that multiplies the normed output element by element (a layer
-    scale), "" for none."""
+    scale), "" for none; ``scalar``: the gain's tensor holds one number for all elements."""
     size: int
     eps: float
     gain_name: str
     scale_name: str = ""
     one_plus: bool = False
     kind: str = "post_norm"
+    scalar: bool = False
 
 
 @dataclass(frozen=True)
@@ -318,12 +364,15 @@ class SwiGLUSpec:
 @dataclass(frozen=True)
 class EmbeddingSpec:
     """h[t] = table[ids[t]] * scale; ``copies`` > 1: [tokens, copies, hidden] with every row that many times
-    (a residual kept as several streams starts with all of them equal)."""
+    (a residual kept as several streams starts with all of them equal).  ``side_width`` > 0: a second table of token
+    rows of that width (tensor ``side_name``) from which the layers' ``token_side`` parts read their columns."""
     vocab_size: int
     hidden_size: int
     kind: str = "embedding"
     scale: float = 1.0
     copies: int = 1
+    side_width: int = 0
+    side_name: str = "side"
 
 
 @dataclass(frozen=True)
@@ -439,6 +488,26 @@ class SandwichLayerSpec:
     ffn_link: object = None
     names: Tuple[Tuple[str, str], ...] = ()
     arrangement: str = "sandwich"
+
+    def prefix(self, part: str) -> str:
+        return dict(self.names).get(part, "")
+
+
+@dataclass(frozen=True)
+class PostLayerSpec:
+    """One block whose sublayers read the residual itself and whose norms stand behind them (``arrangement`` "postnorm"):
+    x <- x + link1(mixer(x)), then (``ffn`` not None) x <- x + link2(ffn(x)), then (``side`` not None) x <- x + link3(side(x)).
+    ``reader`` hands a sublayer the residual (a :class:`NoNormSpec`); the links are norms behind (:class:`PostNormSpec`).
+    ``names`` maps the parts to the prefixes of their tensors."""
+    mixer: object
+    reader: object
+    mixer_link: object
+    ffn: object = None
+    ffn_link: object = None
+    side: object = None
+    side_link: object = None
+    names: Tuple[Tuple[str, str], ...] = ()
+    arrangement: str = "postnorm"
 
     def prefix(self, part: str) -> str:
         return dict(self.names).get(part, "")

@@ -36,6 +36,7 @@
 #include "common.cuh"
 #include "mma_helpers.cuh"
 #include "softcap.cuh"
+#include "distance_bias.cuh"
 #include <cuda.h>
 #include <float.h>
 
@@ -111,7 +112,7 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
                         float* __restrict__ o_part, float* __restrict__ ml_part, const int* __restrict__ page_table,
                         const int* __restrict__ seq_slot, const int* __restrict__ seq_len, int H, int KV, int mpps,
                         int num_pages, int max_chunks, float scale_log2, int window, int* __restrict__ err,
-                        float cap_raw) {
+                        float cap_raw, DistBias bias) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     DecodeSmem& sm = *reinterpret_cast<DecodeSmem*>(smem_raw);
     float* comb = reinterpret_cast<float*>(smem_raw + sizeof(DecodeSmem));
@@ -219,6 +220,11 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
                 int key = key0 + t * 8 + qc * 2 + (e & 1);
                 bool vis = page >= 0 && key < len && key >= first_key;
                 s[t][e] = vis ? s[t][e] * scale_log2 : -FLT_MAX;
+                if (bias.table && vis) {              // a distance bias, after the scale and the cap
+                    const int row = g0 + quad + (e >> 1) * 8;
+                    s[t][e] = fmaf(ri_bias_at(ri_bias_row(bias, kvh * G + (row < G ? row : 0)), bias.len, len - 1 - key),
+                                   1.4426950408889634f, s[t][e]);
+                }
                 mx[e >> 1] = fmaxf(mx[e >> 1], s[t][e]);
             }
         float sum[2] = {0.0f, 0.0f};
@@ -395,6 +401,8 @@ struct StreamArgs {
     int seqs, KV, mpps, num_pages, window, max_pages, parts;
     int* err;
     float cap_raw;          // a soft cap on the scores in unscaled units (cap / scale), 0 for none
+    DistBias bias;          // a distance bias per head on the scores (table null: none)
+    float inv_scale;        // 1 / scale: the bias in unscaled units
     int shared_kv;          // the values are the keys (one pool given as both): a page's tile is copied once and serves as both
 };
 
@@ -727,6 +735,25 @@ attention_decode_stream_kernel(const bf16* __restrict__ q, const __grid_constant
             for (int t = 0; t < 4; t++)
 #pragma unroll
                 for (int e = 0; e < 4; e++) s[t][e] = ri_softcap(s[t][e], a.cap_raw, inv_cap);
+        }
+        if (a.bias.table) {                    // a distance bias (in unscaled units), after the cap and before the mask
+            const int G1 = G - 1;
+            const float* b0 = ri_bias_row(a.bias, cc.kvh * G + min(quad, G1));
+            const float* b1 = ri_bias_row(a.bias, cc.kvh * G + min(quad + 8, G1));
+            const int last = a.bias.len - 1, d0 = cc.len - 1 - key0;          // the distance of the page's first key
+            if (d0 - (AD_PAGE - 1) >= last) {                                 // the whole page lies in the last entry
+                const float f0 = __ldg(b0 + last) * a.inv_scale, f1 = __ldg(b1 + last) * a.inv_scale;
+#pragma unroll
+                for (int t = 0; t < 4; t++)
+#pragma unroll
+                    for (int e = 0; e < 4; e++) s[t][e] += (e >> 1) ? f1 : f0;
+            } else {
+#pragma unroll
+                for (int t = 0; t < 4; t++)
+#pragma unroll
+                    for (int e = 0; e < 4; e++)
+                        s[t][e] = fmaf(ri_bias_at((e >> 1) ? b1 : b0, a.bias.len, d0 - (t * 8 + qc * 2 + (e & 1))), a.inv_scale, s[t][e]);
+            }
         }
         // ---- mask (only the pages at the ends of the visible range need it), maximum, weights ---------------
         if (key0 < cc.first_key || rows < AD_PAGE) {
@@ -1088,14 +1115,17 @@ extern "C" int ri_attention_decode_parts(int max_chunks) {
 // parts = ri_attention_decode_parts(max_chunks).  max_chunks * 128 must cover the longest sequence of the step.
 // sink [H] float32 or null: a learned term per head that joins the softmax's denominator only (the merge adds it).
 // softcap > 0: score <- softcap * tanh(score / softcap) after the scale (0: none; the scale must then be positive).
+// dist_bias [H, bias_len] float32 or null: added to the score by the query's distance to the key (distance_bias.cuh).
 extern "C" int ri_attention_decode_cap(const void* q, const void* k_pool, const void* v_pool, void* out, float* o_part,
                                        float* ml_part, const int* page_table, const int* seq_slot, const int* seq_len,
                                        int seqs, int H, int KV, int Dh, int mpps, int page_size, int num_pages,
                                        int max_chunks, float scale, int window, const float* sink, float softcap,
-                                       int* err_flag, cudaStream_t stream) {
+                                       const float* dist_bias, int bias_len, int* err_flag, cudaStream_t stream) {
     if (seqs == 0) return 0;
     RI_REQUIRE(softcap >= 0.0f && (softcap == 0.0f || scale > 0.0f), "attention_decode: a soft cap %g with scale %g", (double)softcap, (double)scale);
     const float cap_raw = softcap > 0.0f ? softcap / scale : 0.0f;
+    RI_REQUIRE(!dist_bias || bias_len > 0, "attention_decode: a distance bias needs its length");
+    const DistBias bias{dist_bias, bias_len};
     RI_REQUIRE(Dh == AD_DH, "attention_decode: built for head_dim %d, called with %d", AD_DH, Dh);
     RI_REQUIRE(page_size == AD_PAGE, "attention_decode: pages of %d tokens, this kernel needs %d", page_size, AD_PAGE);
     RI_REQUIRE(H > 0 && KV > 0 && H % KV == 0, "attention_decode: %d heads over %d kv heads", H, KV);
@@ -1131,6 +1161,8 @@ extern "C" int ri_attention_decode_cap(const void* q, const void* k_pool, const 
         a.window = window;
         a.err = err_flag;
         a.cap_raw = cap_raw;
+        a.bias = bias;
+        a.inv_scale = 1.0f / scale;
         a.shared_kv = k_pool == v_pool ? 1 : 0;
         // the most runs of ADS_MIN_PAGES pages that the step can have: fewer blocks than SMs, or fewer warps per
         // block (each with a deeper ring), when they do not fill the grid
@@ -1163,7 +1195,7 @@ extern "C" int ri_attention_decode_cap(const void* q, const void* k_pool, const 
     dim3 grid(max_chunks, KV, seqs);
     ri_launch_pdl(attention_decode_kernel, grid, dim3(32 * AD_WARPS), smem, stream,
                   (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, o_part, ml_part, page_table, seq_slot, seq_len,
-                  H, KV, mpps, num_pages, max_chunks, scale * 1.4426950408889634f, window, err_flag, cap_raw);
+                  H, KV, mpps, num_pages, max_chunks, scale * 1.4426950408889634f, window, err_flag, cap_raw, bias);
     RI_CHECK_LAUNCH("attention_decode");
     MergeCut chunks_of_128;
     chunks_of_128.workers = 0;
@@ -1182,7 +1214,8 @@ extern "C" int ri_attention_decode_sink(const void* q, const void* k_pool, const
                                         int max_chunks, float scale, int window, const float* sink, int* err_flag,
                                         cudaStream_t stream) {
     return ri_attention_decode_cap(q, k_pool, v_pool, out, o_part, ml_part, page_table, seq_slot, seq_len, seqs, H, KV, Dh,
-                                   mpps, page_size, num_pages, max_chunks, scale, window, sink, 0.0f, err_flag, stream);
+                                   mpps, page_size, num_pages, max_chunks, scale, window, sink, 0.0f, nullptr, 0,
+                                   err_flag, stream);
 }
 
 extern "C" int ri_attention_decode(const void* q, const void* k_pool, const void* v_pool, void* out, float* o_part,

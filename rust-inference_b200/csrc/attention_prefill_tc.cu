@@ -58,6 +58,7 @@
 #include "common.cuh"
 #include "mma_helpers.cuh"
 #include "softcap.cuh"
+#include "distance_bias.cuh"
 #include <cuda.h>
 #include <float.h>
 
@@ -288,6 +289,8 @@ struct TcWork {
     int seqs, H, KV, mpps, groups_max, n_items, window;
     const float* sink;          // [H] or null: exp(sink[h]) joins head h's softmax denominator, with no key and no value
     float cap_raw;              // a soft cap on the scores in unscaled units (cap / scale), 0 for none
+    DistBias bias;              // a distance bias per head on the scores (table null: none)
+    float inv_scale;            // 1 / scale: the bias in unscaled units
 };
 // The items in the order (group of rows: late ones, which see the most keys, first; sequence; head).  Block c of G
 // takes item k G + c in its round k when k is even and item k G + G - 1 - c when k is odd, so the block that drew
@@ -325,6 +328,8 @@ __device__ __forceinline__ int tc_tile_blocks(const TcItem& it, int t) {
     return t < it.n_tiles ? (t == 0 ? it.n_blocks_0 : it.n_blocks) : 0;
 }
 
+// BIAS: with a distance bias (a variant of its own, so that the others keep their registers)
+template <bool BIAS>
 __global__ void __launch_bounds__(TC_THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                              const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out, const TcWork work,
@@ -576,6 +581,18 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
                     for (int i = 0; i < TC_BN; i++) s[i] = ri_softcap(s[i], work.cap_raw, inv_cap);
                 }
+                if (BIAS) {                                           // a distance bias, after the cap and before the mask
+                    const float* brow = ri_bias_row(work.bias, it.h);
+                    const int last = work.bias.len - 1, d0 = my_pos - kb * TC_BN;          // the distance of the block's first key
+                    if (tile_first - (kb * TC_BN + TC_BN - 1) >= last) {                   // the whole block lies in the last entry
+                        const float far_bias = __ldg(brow + last) * work.inv_scale;
+#pragma unroll
+                        for (int i = 0; i < TC_BN; i++) s[i] += far_bias;
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < TC_BN; i++) s[i] = fmaf(ri_bias_at(brow, work.bias.len, d0 - i), work.inv_scale, s[i]);
+                    }
+                }
                 // a block of keys needs the mask if some query of this tile does not see all of it
                 const bool edge = (kb * TC_BN + TC_BN - 1 > tile_first) || (window != 0 && kb * TC_BN < ri_first_visible(tile_last, window));
                 if (edge) {
@@ -787,10 +804,13 @@ extern "C" int ri_attention_prefill_tc(const void* q, const void* k_pool, const 
                                        const int* page_table, const int* seq_slot, const int* seq_start,
                                        const int* seq_len, int tokens, int seqs, int max_new, int H, int KV, int Dh, int mpps,
                                        int page_size, int num_pages, float scale, int window, const float* sink,
-                                       float softcap, int* err_flag, cudaStream_t stream) {
+                                       float softcap, const float* dist_bias, int bias_len, int* err_flag,
+                                       cudaStream_t stream) {
+    // dist_bias [H, bias_len] float32 or null: added to the score by the query's distance to the key (distance_bias.cuh)
     // softcap > 0: score <- softcap * tanh(score / softcap) after the scale (0: none)
     if (seqs == 0 || max_new == 0 || tokens == 0) return 0;
     RI_REQUIRE(softcap >= 0.0f, "attention_prefill_tc: a soft cap is positive (0: none), got %g", (double)softcap);
+    RI_REQUIRE(!dist_bias || bias_len > 0, "attention_prefill_tc: a distance bias needs its length");
     RI_REQUIRE(Dh == TC_DH, "attention_prefill_tc: built for head_dim %d, called with %d", TC_DH, Dh);
     RI_REQUIRE(page_size == TC_PAGE, "attention_prefill_tc: pages of %d tokens, this kernel needs %d", page_size, TC_PAGE);
     RI_REQUIRE(H > 0 && KV > 0 && H % KV == 0, "attention_prefill_tc: %d heads over %d kv heads", H, KV);
@@ -812,7 +832,8 @@ extern "C" int ri_attention_prefill_tc(const void* q, const void* k_pool, const 
     static bool configured = false;
     static int sms = 0;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC_SMEM_BYTES);
+        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC_SMEM_BYTES);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_prefill_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC_SMEM_BYTES);
         if (e != cudaSuccess) RI_FAIL((int)e, "attention_prefill_tc: %s", cudaGetErrorString(e));
         int dev = 0;
         cudaGetDevice(&dev);
@@ -834,10 +855,17 @@ extern "C" int ri_attention_prefill_tc(const void* q, const void* k_pool, const 
     work.window = window;
     work.sink = sink;
     work.cap_raw = softcap > 0.0f ? softcap / scale : 0.0f;
+    work.bias = DistBias{dist_bias, bias_len};
+    work.inv_scale = 1.0f / scale;
     // one block per SM (the kernel's shared memory allows no second), each taking its items one after the other
     const int blocks = n_items < sms ? (int)n_items : sms;
-    attention_prefill_tc_kernel<<<blocks, TC_THREADS, TC_SMEM_BYTES, stream>>>(
-        map_q, map_k, map_v, (bf16*)out, work, num_pages, scale * 1.4426950408889634f, err_flag);
+    const float scale_log2 = scale * 1.4426950408889634f;
+    if (dist_bias)
+        attention_prefill_tc_kernel<true><<<blocks, TC_THREADS, TC_SMEM_BYTES, stream>>>(map_q, map_k, map_v, (bf16*)out, work,
+                                                                                         num_pages, scale_log2, err_flag);
+    else
+        attention_prefill_tc_kernel<false><<<blocks, TC_THREADS, TC_SMEM_BYTES, stream>>>(map_q, map_k, map_v, (bf16*)out, work,
+                                                                                          num_pages, scale_log2, err_flag);
     RI_CHECK_LAUNCH("attention_prefill_tc");
     return 0;
 }

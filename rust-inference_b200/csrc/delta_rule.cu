@@ -10,6 +10,7 @@
 // `delta_rule_recurrent`: per head h with q/k head h / (H / G), for every new token in order
 //     qn = q / sqrt(sum q^2 + 1e-6) * qscale,   kn = k / sqrt(sum k^2 + 1e-6)
 //     g[d] = exp(-exp(A_log[h]) * softplus(z[h, d] + dt_bias[h, d]))          decay of key channel d
+//            (or one decay per head, g = exp(-exp(A_log[h]) * softplus(z[h] + dt_bias[h])), for all its channels)
 //     beta = sigmoid(b[h])
 //     S[d, j] <- g[d] S[d, j];   u[j] = beta (v[j] - sum_d S[d, j] kn[d]);   S[d, j] <- S[d, j] + kn[d] u[j]
 //     o[j] = sum_d S[d, j] qn[d]                                              (reads the current token's write)
@@ -163,13 +164,14 @@ extern "C" int ri_short_conv(const void* x, long long ld, int col0, const float*
 
 // ---- what the recurrence reads, made ready for all tokens at once ------------------------------------------------------
 // One block per token: q and k of every q/k head become unit vectors in place (q also times qscale), the decays
-// g[h, d] = exp(-exp(A_log[h]) softplus(z[h, d] + dt_bias[h, d])), beta[h] = sigmoid(b[h]) and the products k . q of the
-// unit vectors are written as float32 (`beta` [tokens, H + G]: the betas, then the products).
+// g[h, d] = exp(-exp(A_log[h]) softplus(z[h, d] + dt_bias[h, d])) with d < ddim (ddim = dim, or 1: one decay per head),
+// beta[h] = sigmoid(b[h]) and the products k . q of the unit vectors are written as float32 (`beta` [tokens, H + G]: the
+// betas, then the products).  Row t of z starts ldz elements after row t - 1.
 template <typename T>
 __global__ void __launch_bounds__(128)
 delta_prep_kernel(float* __restrict__ qkv, int C, int q_col, int k_col, const T* __restrict__ proj, long long ld, int b_col,
-                  const T* __restrict__ z, const float* __restrict__ dt_bias, const float* __restrict__ a_log, float qscale,
-                  float* __restrict__ decay, float* __restrict__ beta, int H, int G, int dim) {
+                  const T* __restrict__ z, long long ldz, const float* __restrict__ dt_bias, const float* __restrict__ a_log,
+                  float qscale, float* __restrict__ decay, float* __restrict__ beta, int H, int G, int dim, int ddim) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
@@ -193,9 +195,9 @@ delta_prep_kernel(float* __restrict__ qkv, int C, int q_col, int k_col, const T*
         }
         if (lane == 0) beta[(size_t)t * (H + G) + H + g] = qk * iq * ik;
     }
-    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < H * dim; i += blockDim.x * gridDim.y) {
-        const float rate = expf(a_log[i / dim]);
-        decay[(size_t)t * H * dim + i] = expf(-rate * dr_softplus(ld_f(z + (size_t)t * H * dim + i) + dt_bias[i]));
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < H * ddim; i += blockDim.x * gridDim.y) {
+        const float rate = expf(a_log[i / ddim]);
+        decay[(size_t)t * H * ddim + i] = expf(-rate * dr_softplus(ld_f(z + (size_t)t * ldz + i) + dt_bias[i]));
     }
     for (int h = blockIdx.y * blockDim.x + threadIdx.x; h < H; h += blockDim.x * gridDim.y)
         beta[(size_t)t * (H + G) + h] = 1.0f / (1.0f + expf(-ld_f(proj + (size_t)t * ld + b_col + h)));
@@ -217,7 +219,9 @@ delta_prep_kernel(float* __restrict__ qkv, int C, int q_col, int k_col, const T*
 // The read-out after the write, o = (S' + k u^T)^T q with S' the decayed state, is taken as S'^T q + u (k . q): both
 // sums over d then run over the same S' side by side (their shuffles travel together), and the write S' + k u^T is
 // off the chain to the next token's sums by one multiply-add.
-template <int CH, int SPLIT, int GROUP>
+// SCALAR (one decay per head): the sums run over the undecayed state and are multiplied by the decay afterwards,
+// S'^T k = g (S^T k), so that the decay itself, S' = g S, is off the chain; only its one number per token is staged.
+template <int CH, int SPLIT, int GROUP, bool SCALAR>
 __global__ void __launch_bounds__(DR_THREADS)
 delta_rule_kernel(const float* __restrict__ qkv, int C, int q_col, int k_col, int v_col, const float* __restrict__ decay,
                   const float* __restrict__ beta, float* __restrict__ state, float* __restrict__ o,
@@ -226,9 +230,9 @@ delta_rule_kernel(const float* __restrict__ qkv, int C, int q_col, int k_col, in
     constexpr int DR_BCOLS = DR_THREADS / SPLIT;
     constexpr int PER = (GROUP * DIMC + DR_THREADS - 1) / DR_THREADS;      // staged elements per thread and array
     constexpr int VPER = (GROUP * DR_BCOLS + DR_THREADS - 1) / DR_THREADS;
-    __shared__ __align__(16) float s_g[2][GROUP][DIMC], s_k[2][GROUP][DIMC], s_q[2][GROUP][DIMC];
+    __shared__ __align__(16) float s_g[2][GROUP][SCALAR ? 4 : DIMC], s_k[2][GROUP][DIMC], s_q[2][GROUP][DIMC];
     __shared__ float s_v[2][GROUP][DR_BCOLS], s_beta[2][GROUP], s_kq[2][GROUP];
-    static_assert(2 * GROUP <= DR_THREADS, "a thread per staged beta and per staged product");
+    static_assert(3 * GROUP <= DR_THREADS, "a thread per staged beta, product and decay");
     // (the kernel after this one is let in only when the walk is over, see below)
     const int b = blockIdx.z, h = blockIdx.y;
     const int kvh = h / (H / G);
@@ -252,7 +256,7 @@ delta_rule_kernel(const float* __restrict__ qkv, int C, int q_col, int k_col, in
             const int g = idx / DIMC, d = idx % DIMC, t = base + g;
             rg[e] = rk[e] = rq[e] = 0.0f;
             if (g < GROUP && t < t1 && d < dim) {
-                rg[e] = decay[((size_t)t * H + h) * dim + d];
+                if (!SCALAR) rg[e] = decay[((size_t)t * H + h) * dim + d];
                 rk[e] = qkv[(size_t)t * C + k_col + kvh * dim + d];
                 rq[e] = qkv[(size_t)t * C + q_col + kvh * dim + d];
             }
@@ -266,6 +270,9 @@ delta_rule_kernel(const float* __restrict__ qkv, int C, int q_col, int k_col, in
         if (threadIdx.x < 2 * GROUP) {
             const int g = threadIdx.x % GROUP;
             rb = base + g < t1 ? beta[(size_t)(base + g) * (H + G) + (threadIdx.x < GROUP ? h : H + kvh)] : 0.0f;
+        } else if (SCALAR && threadIdx.x < 3 * GROUP) {
+            const int g = threadIdx.x - 2 * GROUP;
+            rb = base + g < t1 ? decay[(size_t)(base + g) * H + h] : 0.0f;
         }
     };
     auto store = [&](int buf) {
@@ -273,7 +280,7 @@ delta_rule_kernel(const float* __restrict__ qkv, int C, int q_col, int k_col, in
         for (int e = 0; e < PER; e++) {
             const int idx = threadIdx.x + e * DR_THREADS;
             if (idx < GROUP * DIMC) {
-                (&s_g[buf][0][0])[idx] = rg[e];
+                if (!SCALAR) (&s_g[buf][0][0])[idx] = rg[e];
                 (&s_k[buf][0][0])[idx] = rk[e];
                 (&s_q[buf][0][0])[idx] = rq[e];
             }
@@ -285,6 +292,7 @@ delta_rule_kernel(const float* __restrict__ qkv, int C, int q_col, int k_col, in
         }
         if (threadIdx.x < GROUP) s_beta[buf][threadIdx.x] = rb;
         else if (threadIdx.x < 2 * GROUP) s_kq[buf][threadIdx.x - GROUP] = rb;
+        else if (SCALAR && threadIdx.x < 3 * GROUP) s_g[buf][threadIdx.x - 2 * GROUP][0] = rb;
     };
     fetch(t0);
     int buf = 0;
@@ -299,14 +307,14 @@ delta_rule_kernel(const float* __restrict__ qkv, int C, int q_col, int k_col, in
 #pragma unroll
             for (int i = 0; i < CH; i += 4) {
                 const int at = 4 * SPLIT * (i / 4) + 4 * part;
-                const float4 gg = *reinterpret_cast<const float4*>(&s_g[buf][g][at]);
+                const float4 gg = SCALAR ? make_float4(1.0f, 1.0f, 1.0f, 1.0f) : *reinterpret_cast<const float4*>(&s_g[buf][g][SCALAR ? 0 : at]);
                 const float4 kk = *reinterpret_cast<const float4*>(&s_k[buf][g][at]);
                 const float4 qq = *reinterpret_cast<const float4*>(&s_q[buf][g][at]);
                 kr[i / 4] = kk;
-                S[i] *= gg.x;     p[0] = fmaf(S[i], kk.x, p[0]);     a[0] = fmaf(S[i], qq.x, a[0]);
-                S[i + 1] *= gg.y; p[1] = fmaf(S[i + 1], kk.y, p[1]); a[1] = fmaf(S[i + 1], qq.y, a[1]);
-                S[i + 2] *= gg.z; p[2] = fmaf(S[i + 2], kk.z, p[2]); a[2] = fmaf(S[i + 2], qq.z, a[2]);
-                S[i + 3] *= gg.w; p[3] = fmaf(S[i + 3], kk.w, p[3]); a[3] = fmaf(S[i + 3], qq.w, a[3]);
+                if (!SCALAR) S[i] *= gg.x;     p[0] = fmaf(S[i], kk.x, p[0]);     a[0] = fmaf(S[i], qq.x, a[0]);
+                if (!SCALAR) S[i + 1] *= gg.y; p[1] = fmaf(S[i + 1], kk.y, p[1]); a[1] = fmaf(S[i + 1], qq.y, a[1]);
+                if (!SCALAR) S[i + 2] *= gg.z; p[2] = fmaf(S[i + 2], kk.z, p[2]); a[2] = fmaf(S[i + 2], qq.z, a[2]);
+                if (!SCALAR) S[i + 3] *= gg.w; p[3] = fmaf(S[i + 3], kk.w, p[3]); a[3] = fmaf(S[i + 3], qq.w, a[3]);
             }
             float pred = (p[0] + p[1]) + (p[2] + p[3]);
             float acc = (a[0] + a[1]) + (a[2] + a[3]);
@@ -315,7 +323,13 @@ delta_rule_kernel(const float* __restrict__ qkv, int C, int q_col, int k_col, in
                 pred += __shfl_xor_sync(0xffffffffu, pred, sh);
                 acc += __shfl_xor_sync(0xffffffffu, acc, sh);
             }
-            const float u = s_beta[buf][g] * (s_v[buf][g][col] - pred);
+            const float gs = SCALAR ? s_g[buf][g][0] : 1.0f;
+            const float u = s_beta[buf][g] * (SCALAR ? fmaf(-gs, pred, s_v[buf][g][col]) : s_v[buf][g][col] - pred);
+            if (SCALAR) {
+                acc *= gs;
+#pragma unroll
+                for (int i = 0; i < CH; i++) S[i] *= gs;
+            }
 #pragma unroll
             for (int i = 0; i < CH; i += 4) {
                 S[i] = fmaf(kr[i / 4].x, u, S[i]);
@@ -340,44 +354,52 @@ delta_rule_kernel(const float* __restrict__ qkv, int C, int q_col, int k_col, in
 
 // qkv [tokens, C] float32 (the convolution's output; its q and k columns are made unit vectors in place): q of q/k head g
 // at columns q_col + g dim .., k at k_col + g dim .., v of head h at v_col + h vdim ..;  proj [tokens, ld] (compute type):
-// beta's logit of head h at column b_col + h;  z [tokens, H dim] (compute type): the decay's projection, dt_bias [H dim]
-// and a_log [H] float32;  decay [tokens, H dim] and beta [tokens, H + G]: float32 scratch that this call fills;
+// beta's logit of head h at column b_col + h;  z [tokens, H ddim] (compute type, rows ldz apart): the decay's projection,
+// dt_bias [H ddim] and a_log [H] float32, ddim = dim (a decay per key channel) or 1 (one per head);  decay [tokens, H ddim] and beta [tokens, H + G]: float32 scratch that this call fills;
 // state [slots, H, dim, vdim] float32, updated in place;  o [tokens, H, vdim] float32.
 extern "C" int ri_delta_rule_recurrent(float* qkv, int C, int q_col, int k_col, int v_col, const void* proj, long long ld,
-                                       int b_col, const void* z, const float* dt_bias, const float* a_log, float qscale,
+                                       int b_col, const void* z, long long ldz, int ddim, const float* dt_bias,
+                                       const float* a_log, float qscale,
                                        float* decay, float* beta, float* state, float* o, const int* seq_slot,
                                        const int* seq_start, int tokens, int seqs, int H, int G, int dim, int vdim,
                                        int single, int dtype, cudaStream_t stream) {
     if (seqs == 0 || tokens == 0) return 0;
     RI_REQUIRE(seqs > 0 && tokens > 0 && H > 0 && G > 0 && H % G == 0 && dim > 0 && vdim > 0, "delta_rule_recurrent: bad sizes");
     RI_REQUIRE(seqs <= 65535 && H <= 65535, "delta_rule_recurrent: %d sequences, %d heads: too many for one launch", seqs, H);
+    RI_REQUIRE(ddim == dim || ddim == 1, "delta_rule_recurrent: %d decays per head of %d key channels", ddim, dim);
     RI_REQUIRE(dim <= 512, "delta_rule_recurrent: %d key channels per head (up to 512 are built)", dim);
     const int spread = tokens >= 256 ? 1 : (H * dim + 127) / 128 > 16 ? 16 : (H * dim + 127) / 128;
     const dim3 pgrid(tokens, spread);
     if (dtype == RI_DTYPE_F32)
         ri_launch_pdl(delta_prep_kernel<float>, pgrid, dim3(128), 0, stream, qkv, C, q_col, k_col, (const float*)proj, ld,
-                      b_col, (const float*)z, dt_bias, a_log, qscale, decay, beta, H, G, dim);
+                      b_col, (const float*)z, ldz, dt_bias, a_log, qscale, decay, beta, H, G, dim, ddim);
     else if (dtype == RI_DTYPE_BF16)
         ri_launch_pdl(delta_prep_kernel<__nv_bfloat16>, pgrid, dim3(128), 0, stream, qkv, C, q_col, k_col,
-                      (const __nv_bfloat16*)proj, ld, b_col, (const __nv_bfloat16*)z, dt_bias, a_log, qscale, decay, beta, H, G, dim);
+                      (const __nv_bfloat16*)proj, ld, b_col, (const __nv_bfloat16*)z, ldz, dt_bias, a_log, qscale, decay, beta, H,
+                      G, dim, ddim);
     else RI_FAIL(-1, "delta_rule_recurrent: unknown dtype %d", dtype);
     RI_CHECK_LAUNCH("delta_prep");
     // The recurrence kernel is launched the ordinary way, not as a dependent launch: its few long-lived blocks (a chain of
     // dependent instructions, one warp per scheduler) must spread one per SM, and blocks that come in while the kernel
     // before still holds most SMs pile up on the first SMs that get free and stay there (2,048 tokens of 8 heads of
     // 128 x 128: 0.97 ms as a dependent launch, 0.59 ms as an ordinary one).
-#define DR_GO(CH, SPLIT, GROUP)                                                                                          \
+#define DR_GO(CH, SPLIT, GROUP, SC)                                                                                        \
     do {                                                                                                                 \
         const int bcols = DR_THREADS / SPLIT;                                                                            \
         const dim3 grid((vdim + bcols - 1) / bcols, H, seqs);                                                            \
-        delta_rule_kernel<CH, SPLIT, GROUP><<<grid, dim3(DR_THREADS), 0, stream>>>(                                       \
+        delta_rule_kernel<CH, SPLIT, GROUP, SC><<<grid, dim3(DR_THREADS), 0, stream>>>(                                       \
             (const float*)qkv, C, q_col, k_col, v_col, (const float*)decay, (const float*)beta, state, o, seq_slot,      \
             seq_start, H, G, dim, vdim);                                                                                 \
     } while (0)
 #define DR_BY_GROUP(CH, SPLIT, GROUP)                                                                                    \
     do {                                                                                                                 \
-        if (single) DR_GO(CH, SPLIT, 1);                                                                                 \
-        else DR_GO(CH, SPLIT, GROUP);                                                                                    \
+        if (ddim == 1 && dim > 1) {                                                                                      \
+            if (single) DR_GO(CH, SPLIT, 1, true);                                                                       \
+            else DR_GO(CH, SPLIT, GROUP, true);                                                                          \
+        } else {                                                                                                         \
+            if (single) DR_GO(CH, SPLIT, 1, false);                                                                      \
+            else DR_GO(CH, SPLIT, GROUP, false);                                                                         \
+        }                                                                                                                \
     } while (0)
     if (dim <= 16) DR_BY_GROUP(4, 4, 16);
     else if (dim <= 32) DR_BY_GROUP(4, 8, 16);

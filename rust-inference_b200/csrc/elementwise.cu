@@ -558,6 +558,67 @@ extern "C" int ri_activation(const void* x, void* out, long long n, int kind, in
 }
 
 // ---------------------------------------------------------------------------
+// An activation times a token's row of a table:
+//   out[t, c] = act(x[t, c]) * table[ids[t]][c],  c < dim;  float32, rounded once
+// x, out [tokens, dim] dense; table rows are `ldt` elements apart (one layer's columns of a table that all layers share).
+// A token outside the table: error word 1, its row becomes zeros.
+// ---------------------------------------------------------------------------
+template <typename T>
+__global__ void act_rows_kernel(const T* __restrict__ x, const int* __restrict__ ids, const T* __restrict__ table, long long ldt,
+                                T* __restrict__ out, int dim, size_t total, int vocab, int kind, int* __restrict__ err) {
+    pdl_trigger();
+    pdl_wait();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+        const size_t t = i / dim;
+        const int c = (int)(i - t * dim), id = ids[t];
+        const bool ok = id >= 0 && id < vocab;
+        if (!ok) atomicExch(err, 1);
+        st_f(out + i, ok ? act_of(ld_f(x + i), kind) * ld_f(table + (size_t)id * ldt + c) : 0.0f);
+    }
+}
+
+// eight neighbouring elements per thread
+template <typename T>
+__global__ void act_rows_vec8_kernel(const T* __restrict__ x, const int* __restrict__ ids, const T* __restrict__ table, long long ldt,
+                                     T* __restrict__ out, int dim8, size_t total8, int vocab, int kind, int* __restrict__ err) {
+    pdl_trigger();
+    pdl_wait();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total8; i += (size_t)gridDim.x * blockDim.x) {
+        const size_t t = i / dim8;
+        const int c = (int)(i - t * dim8) * 8, id = ids[t];
+        const bool ok = id >= 0 && id < vocab;
+        if (!ok) atomicExch(err, 1);
+        Pack8<T> a, e, o;
+        a.load(x + 8 * i);
+        e.load(table + (size_t)(ok ? id : 0) * ldt + c);
+#pragma unroll
+        for (int j = 0; j < 4; j++)
+            o.set2(j, ok ? act_of(a.get(2 * j), kind) * e.get(2 * j) : 0.0f, ok ? act_of(a.get(2 * j + 1), kind) * e.get(2 * j + 1) : 0.0f);
+        o.store(out + 8 * i);
+    }
+}
+
+extern "C" int ri_act_rows(const void* x, const int* ids, const void* table, long long ldt, void* out, int tokens, int dim, int vocab,
+                           int kind, int dtype, int* err_flag, cudaStream_t stream) {
+    if (tokens == 0) return 0;
+    RI_REQUIRE(tokens > 0 && dim > 0 && vocab > 0 && ldt >= dim && kind >= RI_ACT_RELU2 && kind <= RI_ACT_GELU_ERF,
+               "act_rows: bad arguments tokens=%d dim=%d kind=%d", tokens, dim, kind);
+    RI_REQUIRE(dtype == RI_DTYPE_F32 || dtype == RI_DTYPE_BF16, "act_rows: unknown dtype %d", dtype);
+    const bool vec = dim % 8 == 0 && ldt % 8 == 0 && (((uintptr_t)x | (uintptr_t)out | (uintptr_t)table) & 15) == 0;
+    const size_t total = (size_t)tokens * dim / (vec ? 8 : 1);
+    const unsigned blocks = (unsigned)((total + 127) / 128 < 148 * 16 ? (total + 127) / 128 : 148 * 16);
+#define AR_GO(K, T, D) ri_launch_pdl(K<T>, dim3(blocks), dim3(128), 0, stream, (const T*)x, ids, (const T*)table, ldt, (T*)out, D, total, vocab, kind, err_flag)
+    if (dtype == RI_DTYPE_F32) {
+        if (vec) AR_GO(act_rows_vec8_kernel, float, dim / 8); else AR_GO(act_rows_kernel, float, dim);
+    } else {
+        if (vec) AR_GO(act_rows_vec8_kernel, __nv_bfloat16, dim / 8); else AR_GO(act_rows_kernel, __nv_bfloat16, dim);
+    }
+#undef AR_GO
+    RI_CHECK_LAUNCH("act_rows");
+    return 0;
+}
+
+// ---------------------------------------------------------------------------
 // Gates on the heads of a mixer's output, in place:
 //   x[t, h, j] *= f(g[t, per_head ? h : h * width + j]),  f: 0 sigmoid, 1 silu
 // x [tokens, heads, width] is dense; g is a block of columns of a wider matrix (row pitch ldg).

@@ -81,6 +81,12 @@ struct __align__(1024) SkinnySmem {
 // constants of the gate function 3 (clamped swish): g = min(g, limit), u = clamp(u, -limit, limit), g sigmoid(alpha g) (u + 1)
 struct SkGate {
     float limit, alpha;
+    // rows (without SWIGLU; ids null: none): after the activation output n of token t is multiplied by rows[ids[t] * ld + n],
+    // a token's row of a table of `vocab` rows (an id outside: error 1, the output is 0)
+    const int* ids = nullptr;
+    const bf16* rows = nullptr;
+    long long ld = 0;
+    int vocab = 0;
 };
 
 template <int NT, typename OutT, bool SWIGLU, int STAGES>
@@ -229,6 +235,12 @@ linear_skinny_kernel(const bf16* __restrict__ x, const __grid_constant__ CUtenso
             } else if (act == 3) {
                 v = 0.5f * v * (1.0f + erff(v * 0.7071067811865476f));
             }
+            if (gate.ids) {
+                const int id = gate.ids[tok];
+                const bool ok = id >= 0 && id < gate.vocab;
+                if (!ok) atomicExch(err, 1);
+                v = ok ? v * ld_f(gate.rows + (size_t)id * gate.ld + n0 + row) : 0.0f;
+            }
             st_f(y + (size_t)tok * N + n0 + row, v);
         }
     }
@@ -354,6 +366,22 @@ extern "C" int ri_linear_skinny_gated_with(const void* x, const void* w, void* y
     const SkGate g{limit, alpha};
     const int rc = M <= 8 ? launch_skinny<1, bf16, true>(x, w, y, M, N, K, gate, err_flag, stream, g)
                           : launch_skinny<2, bf16, true>(x, w, y, M, N, K, gate, err_flag, stream, g);
+    if (rc) return rc;
+    RI_CHECK_LAUNCH("linear_skinny");
+    return 0;
+}
+
+// y [M, N] = act(x W^T)[t, n] * rows[ids[t] * ld + n] (bfloat16): an activation and a token's row of a table in the epilogue
+extern "C" int ri_linear_skinny_act_rows(const void* x, const void* w, void* y, int M, int N, int K, int act, const int* ids,
+                                         const void* rows, long long ld, int vocab, int* err_flag, cudaStream_t stream) {
+    if (M == 0 || N == 0) return 0;
+    RI_REQUIRE(M > 0 && M <= 16 && N > 0 && K > 0 && K % 8 == 0 && act >= 0 && act <= 3, "linear_skinny: bad sizes M=%d N=%d K=%d act=%d", M, N, K, act);
+    RI_REQUIRE(ids && rows && ld >= N && vocab > 0, "linear_skinny: bad table of rows");
+    RI_REQUIRE((((uintptr_t)x | (uintptr_t)w) & 15) == 0, "linear_skinny: x and w must be 16-byte aligned");
+    SkGate g{0.0f, 0.0f};
+    g.ids = ids; g.rows = (const bf16*)rows; g.ld = ld; g.vocab = vocab;
+    const int rc = M <= 8 ? launch_skinny<1, bf16, false>(x, w, y, M, N, K, act, err_flag, stream, g)
+                          : launch_skinny<2, bf16, false>(x, w, y, M, N, K, act, err_flag, stream, g);
     if (rc) return rc;
     RI_CHECK_LAUNCH("linear_skinny");
     return 0;

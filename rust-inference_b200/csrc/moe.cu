@@ -18,6 +18,7 @@
 //               replayed from a graph).
 // `moe_combine` y[t] = sum_j w[t, j] (choice j an identity expert ? x[t] : pair_out[t top + j]) (+ extra[t]),
 //               j ascending, float32, rounded once.
+// Without a router, a table names every token id's experts (`ri_moe_plan_table`) and the weights are equal.
 #include "common.cuh"
 #include "mma_helpers.cuh"
 
@@ -297,9 +298,18 @@ extern "C" int ri_moe_route_rule(const void* x, const float* router, const float
 
 // ---- the plan ---------------------------------------------------------------------------------------------------------
 // meta[0] = number of tiles, meta[1] = number of rows in perm.  tiles [max_tiles][3].
+// With a `table` [vocab, top] of experts by token id (no router) the pairs' experts are looked up here, idx[t top + j] =
+// table[ids[t]][j], and written to idx_out for whoever reads the choice later.
+struct MoeTable {
+    const int* ids;
+    const int* table;            // null: idx holds the choice
+    int vocab, top;
+    int* idx_out;
+    int* err;
+};
 __global__ void __launch_bounds__(1024)
-moe_plan_kernel(const int* __restrict__ idx, int* __restrict__ perm, int* __restrict__ tiles, int* __restrict__ meta,
-                int pairs, int E, int max_tiles, int bm) {
+moe_plan_kernel(const int* idx, int* __restrict__ perm, int* __restrict__ tiles, int* __restrict__ meta,
+                int pairs, int E, int max_tiles, int bm, MoeTable by_id) {
     extern __shared__ int plan_sm[];                  // counts [E], offsets [E + 1], cursors [E]
     int* counts = plan_sm;
     int* offsets = counts + E;
@@ -308,7 +318,18 @@ moe_plan_kernel(const int* __restrict__ idx, int* __restrict__ perm, int* __rest
     for (int e = threadIdx.x; e < E; e += blockDim.x) counts[e] = cursor[e] = 0;
     pdl_wait();
     __syncthreads();
+    if (by_id.table) idx = by_id.idx_out;             // (a thread reads back only what it wrote itself)
     for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
+        if (by_id.table) {
+            const int t = p / by_id.top, id = by_id.ids[t];
+            int chosen = -1;
+            if (id >= 0 && id < by_id.vocab) chosen = by_id.table[(size_t)id * by_id.top + (p - t * by_id.top)];
+            if (chosen < 0 || chosen >= E) {
+                atomicExch(by_id.err, id >= 0 && id < by_id.vocab ? 8 : 1);
+                chosen = -1;
+            }
+            by_id.idx_out[p] = chosen;
+        }
         const int e = idx[p];
         if (e >= 0 && e < E) atomicAdd(&counts[e], 1);
     }
@@ -346,7 +367,25 @@ extern "C" int ri_moe_plan(const int* idx, int* perm, int* tiles, int* meta, int
     RI_REQUIRE(pairs > 0 && E > 0 && max_tiles >= ri_moe_max_tiles(pairs, E, bm), "moe_plan: bad sizes");
     const size_t smem = (size_t)(3 * E + 1) * sizeof(int);
     RI_REQUIRE(smem <= 48 * 1024, "moe_plan: %d experts (up to 4095 are built)", E);
-    ri_launch_pdl(moe_plan_kernel, dim3(1), dim3(1024), smem, stream, idx, perm, tiles, meta, pairs, E, max_tiles, bm);
+    ri_launch_pdl(moe_plan_kernel, dim3(1), dim3(1024), smem, stream, idx, perm, tiles, meta, pairs, E, max_tiles, bm,
+                  MoeTable{nullptr, nullptr, 0, 0, nullptr, nullptr});
+    RI_CHECK_LAUNCH("moe_plan");
+    return 0;
+}
+
+// The plan of a step whose experts a table names: ids [tokens] int32, table [vocab, top] int32; idx [tokens, top] gets the
+// choice.  A token id outside the table: error word 1; an expert that does not exist: error word 8 (the pair is left out).
+extern "C" int ri_moe_plan_table(const int* ids, const int* table, int vocab, int top, int* idx, int* perm, int* tiles, int* meta,
+                                 int tokens, int E, int max_tiles, int bm, int* err_flag, cudaStream_t stream) {
+    if (tokens == 0) return 0;
+    RI_REQUIRE(bm == MOE_BM || bm == MOE_BM_WIDE, "moe_plan: tiles of %d rows are not built", bm);
+    RI_REQUIRE(tokens > 0 && top > 0 && vocab > 0 && (long long)tokens * top < (1ll << 31), "moe_plan: bad sizes");
+    const int pairs = tokens * top;
+    RI_REQUIRE(E > 0 && max_tiles >= ri_moe_max_tiles(pairs, E, bm), "moe_plan: bad sizes");
+    const size_t smem = (size_t)(3 * E + 1) * sizeof(int);
+    RI_REQUIRE(smem <= 48 * 1024, "moe_plan: %d experts (up to 4095 are built)", E);
+    ri_launch_pdl(moe_plan_kernel, dim3(1), dim3(1024), smem, stream, (const int*)nullptr, perm, tiles, meta, pairs, E, max_tiles,
+                  bm, MoeTable{ids, table, vocab, top, idx, err_flag});
     RI_CHECK_LAUNCH("moe_plan");
     return 0;
 }
@@ -667,18 +706,20 @@ moe_combine_kernel(const float* __restrict__ pair_out, const int* __restrict__ i
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
+    const float equal = 1.0f / (float)top;               // every choice's weight where none are given
     for (int d = blockIdx.y * blockDim.x + threadIdx.x; d < D; d += gridDim.y * blockDim.x) {
         float acc = 0.0f;
         for (int j = 0; j < top; j++) {
-            const int e = idx[(size_t)t * top + j];
+            const int e = idx ? idx[(size_t)t * top + j] : 0;
             const float v = (e >= E) ? ld_f(x + (size_t)t * D + d) : pair_out[((size_t)t * top + j) * D + d];
-            acc = fmaf(weight[(size_t)t * top + j], v, acc);
+            acc = fmaf(weight ? weight[(size_t)t * top + j] : equal, v, acc);
         }
         if (extra) acc += ld_f(extra + (size_t)t * D + d);
         st_f(y + (size_t)t * D + d, acc);
     }
 }
 
+// weight null: every choice has weight 1 / top; idx null: no choice is an identity expert (x is not read)
 extern "C" int ri_moe_combine(const float* pair_out, const int* idx, const float* weight, const void* x, const void* extra,
                               void* y, int tokens, int D, int top, int E, int dtype, cudaStream_t stream) {
     if (tokens == 0) return 0;

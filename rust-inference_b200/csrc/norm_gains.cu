@@ -91,6 +91,8 @@ __global__ void __launch_bounds__(512) norm_gains_kernel(NgArgs a) {
     const T* y2 = (a.y1 && a.y2) ? (const T*)a.y2 + r * dim : nullptr;
     const bool changes = y1 || trow || a.vec;
     const bool post = y1 && a.post_gain;
+    // without a gain nothing is normed: the new residual itself, in the compute type, for whoever reads it next
+    T* copy = a.gain1 || !a.out1 ? nullptr : (T*)a.out1 + (size_t)blockIdx.x * a.out_pitch;
     float sum = 0.0f;
     float pinv = 1.0f;
     if (post) {
@@ -144,6 +146,10 @@ __global__ void __launch_bounds__(512) norm_gains_kernel(NgArgs a) {
                 if (a.vec) { x.x = x.x + vv.x; x.y = x.y + vv.y; x.z = x.z + vv.z; x.w = x.w + vv.w; }
                 if (a.write_back) ng_st4(rp + 4 * i, x);
             }
+            if (copy) {                                             // nothing is normed: see below
+                ng_st4(copy + 4 * i, x);
+                continue;
+            }
             *reinterpret_cast<float4*>(ng_row + 4 * i) = x;
             sum += (x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w);
         }
@@ -159,19 +165,15 @@ __global__ void __launch_bounds__(512) norm_gains_kernel(NgArgs a) {
                 }
                 if (a.write_back) rp[i] = x;
             }
+            if (copy) {
+                st_f(copy + i, x);
+                continue;
+            }
             ng_row[i] = x;
             sum += x * x;
         }
     }
-    if (!a.gain1) {
-        // nothing is normed: the new residual itself, in the compute type, for whoever reads it next
-        if (a.out1) {
-            __syncthreads();
-            T* oc = (T*)a.out1 + (size_t)blockIdx.x * a.out_pitch;
-            for (int i = threadIdx.x; i < dim; i += blockDim.x) st_f(oc + i, ng_row[i]);
-        }
-        return;
-    }
+    if (!a.gain1) return;
     const float inv = 1.0f / sqrtf(block_sum(sum, red) / (float)dim + a.eps);
     T* o1 = (T*)a.out1 + (size_t)blockIdx.x * dim;
     T* o2 = a.out2 ? (T*)a.out2 + (size_t)blockIdx.x * dim : nullptr;
@@ -216,7 +218,7 @@ extern "C" int ri_norm_gains_post(float* resid, const void* y1, const float* w1,
     RI_REQUIRE(dtype == RI_DTYPE_F32 || dtype == RI_DTYPE_BF16, "norm_gains: unknown dtype %d", dtype);
     RI_REQUIRE(y1 || !y2, "norm_gains: pending outputs are given first, second");
     RI_REQUIRE((gain2 == nullptr) == (out2 == nullptr), "norm_gains: a second gain and a second output go together");
-    RI_REQUIRE(gain1 || (!gain2 && !next_w), "norm_gains: without a first gain nothing is normed");
+    RI_REQUIRE(gain1 || !gain2, "norm_gains: a second gain without a first");
     RI_REQUIRE(gain1 ? out1 != nullptr : (!out1 || out_pitch >= dim), "norm_gains: bad output for %d columns", dim);
     RI_REQUIRE(!post_gain || y1, "norm_gains: a norm behind the sublayer needs its output");
     RI_REQUIRE(!ids || (table && vocab > 0), "norm_gains: token ids need the table");
@@ -241,7 +243,8 @@ extern "C" int ri_norm_gains_post(float* resid, const void* y1, const float* w1,
     }
     const uintptr_t unit = dtype == RI_DTYPE_F32 ? 15 : 7;
     const bool vec4 = dim % 4 == 0 && (((uintptr_t)resid | (uintptr_t)gain1 | (uintptr_t)gain2 | (uintptr_t)vec | (uintptr_t)post_gain) & 15) == 0 &&
-                      (((uintptr_t)y1 | (uintptr_t)y2 | (uintptr_t)table | (uintptr_t)out1 | (uintptr_t)out2) & unit) == 0;
+                      (((uintptr_t)y1 | (uintptr_t)y2 | (uintptr_t)table | (uintptr_t)out1 | (uintptr_t)out2) & unit) == 0 &&
+                      (gain1 || out_pitch % 4 == 0);
     // by the row length alone: the order of a row's additions must not depend on how many rows the step has
     int threads;
     if (vec4) {

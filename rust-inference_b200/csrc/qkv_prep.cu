@@ -15,7 +15,9 @@
 //     a' = a c - b s,  b' = b c + a s;
 // then, with `unit`, the head is divided by its root mean square over its Dk true elements:
 //     x' / sqrt(sum(x'^2) / Dk + eps)                    (no gain);
-// q goes to q_out, k to the token's place in its page.  v heads get their bias and are stored.  All of it float32.
+// and q heads are multiplied by the position's factor, q_factor[pos] (float32 [factor_rows], null: none);
+// q goes to q_out, k to the token's place in its page.  v heads get their bias, are divided by their root mean square
+// over their Dv true elements with `unit_v` (eps as for `unit`, no gain), and are stored.  All of it float32.
 #include "common.cuh"
 
 #define QP_WARPS 4
@@ -31,6 +33,8 @@ struct QpArgs {
     const float2* rope;
     int rope_rows, rot, pairs, unit;
     float eps;
+    const float* q_factor;
+    int factor_rows, unit_v, Dv;
     const float *q_gain, *k_gain;
     int norm;
     float norm_eps;
@@ -85,7 +89,8 @@ __global__ void qkv_prep_kernel(QpArgs a) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int pos = a.tok_pos[t];
     const int page = qp_page(a, t, pos);
-    const bool rope_ok = !a.rope || (pos >= 0 && pos < a.rope_rows);
+    const bool rope_ok = (!a.rope || (pos >= 0 && pos < a.rope_rows)) && (!a.q_factor || (pos >= 0 && pos < a.factor_rows));
+    const float qf = a.q_factor && rope_ok ? a.q_factor[pos] : 1.0f;
     pdl_wait();
     if (!rope_ok) {
         if (threadIdx.x == 0) atomicExch(a.err, 3);
@@ -112,7 +117,13 @@ __global__ void qkv_prep_kernel(QpArgs a) {
         for (int d = lane; d < Dp; d += 32) x[d] = ld_f(row + col + d) + (a.bias ? a.bias[col + d] : 0.0f);
         __syncwarp();
         if (which == 2) {
-            for (int d = lane; d < Dp; d += 32) st_f(dst + d, x[d]);
+            float vinv = 1.0f;
+            if (a.unit_v) {
+                float ss = 0.0f;
+                for (int d = lane; d < Dp; d += 32) ss += x[d] * x[d];
+                vinv = 1.0f / sqrtf(warp_sum(ss) / (float)a.Dv + a.eps);
+            }
+            for (int d = lane; d < Dp; d += 32) st_f(dst + d, x[d] * vinv);
             __syncwarp();
             continue;
         }
@@ -146,6 +157,7 @@ __global__ void qkv_prep_kernel(QpArgs a) {
             for (int d = lane; d < Dp; d += 32) ss += x[d] * x[d];
             inv = 1.0f / sqrtf(warp_sum(ss) / (float)a.Dk + a.eps);
         }
+        if (which == 0) inv *= qf;
         for (int d = lane; d < Dp; d += 32) st_f(dst + d, x[d] * inv);
         __syncwarp();
     }
@@ -232,7 +244,8 @@ __global__ void qkv_prep_vec_kernel(QpArgs a, int group) {
     const bool live_lane = d0 < Dp;
     const int pos = a.tok_pos[t];
     const int page = qp_page(a, t, pos);
-    const bool rope_ok = !a.rope || (pos >= 0 && pos < a.rope_rows);
+    const bool rope_ok = (!a.rope || (pos >= 0 && pos < a.rope_rows)) && (!a.q_factor || (pos >= 0 && pos < a.factor_rows));
+    const float qf = a.q_factor && rope_ok ? a.q_factor[pos] : 1.0f;
     // the angles of this lane's four pairs and its share of the bias do not depend on the kernel in front
     float cs_c[4], cs_s[4];
 #pragma unroll
@@ -335,39 +348,35 @@ __global__ void qkv_prep_vec_kernel(QpArgs a, int group) {
                 x[2 * j + 1] = v * cs_c[j] + u * cs_s[j];
             }
         }
-        if (a.unit) {
+        float inv = which == 0 ? qf : 1.0f;
+        if (a.unit || a.unit_v) {
             float ss = 0.0f;
 #pragma unroll
             for (int j = 0; j < 8; j++) ss += x[j] * x[j];
             for (int o = group >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-            if (which < 2) {
-                const float inv = 1.0f / sqrtf(ss / (float)a.Dk + a.eps);
-#pragma unroll
-                for (int j = 0; j < 8; j++) x[j] *= inv;
-            }
+            if (which < 2 ? a.unit : a.unit_v) inv = 1.0f / sqrtf(ss / (float)(which < 2 ? a.Dk : a.Dv) + a.eps) * inv;
         }
+#pragma unroll
+        for (int j = 0; j < 8; j++) x[j] *= inv;
         if (dst) Qp8<T>::store(dst, x);
     }
 }
 
-extern "C" int ri_qkv_prep(const void* proj, long long ld, int q_col, int k_col, int v_col, const float* bias, void* q_out,
-                           void* k_pool, void* v_pool, const int* page_table, const int* tok_seq, const int* tok_pos,
-                           const int* seq_slot, const float* rope_table, int rope_rows, int rot, int pairs, int unit,
-                           float eps, int tokens, int H, int KV, int Dp, int Dk, int mpps, int page_size, int num_pages,
-                           int write_kv, int dtype, int* err_flag, cudaStream_t stream);
-
-// The same with a norm of q and k heads before the rotation: norm 1 per head (gains [Dp]), 2 over all heads of the
-// token at once (gains [H, Dp] and [KV, Dp]); 0: none.
+// norm: of q and k heads before the rotation, 1 per head (gains [Dp]), 2 over all heads of the token at once (gains [H, Dp]
+// and [KV, Dp]), 0 none.  q_factor [factor_rows] float32 or null: by the token's position, on the q heads.  unit_v: v heads
+// are divided by their root mean square over Dv elements.
 extern "C" int ri_qkv_prep_norm(const void* proj, long long ld, int q_col, int k_col, int v_col, const float* bias, void* q_out,
                                 void* k_pool, void* v_pool, const int* page_table, const int* tok_seq, const int* tok_pos,
                                 const int* seq_slot, const float* rope_table, int rope_rows, int rot, int pairs, int unit,
-                                float eps, const float* q_gain, const float* k_gain, int norm, float norm_eps, int tokens,
-                                int H, int KV, int Dp, int Dk, int mpps, int page_size, int num_pages, int write_kv,
+                                float eps, const float* q_gain, const float* k_gain, int norm, float norm_eps,
+                                const float* q_factor, int factor_rows, int unit_v, int Dv, int tokens, int H, int KV, int Dp,
+                                int Dk, int mpps, int page_size, int num_pages, int write_kv,
                                 int dtype, int* err_flag, cudaStream_t stream) {
     if (tokens == 0) return 0;
     RI_REQUIRE(norm >= 0 && norm <= 2, "qkv_prep: norm %d", norm);
     RI_REQUIRE(!norm || ((q_gain || !H) && (k_gain || !KV)), "qkv_prep: a norm needs its gains");
     RI_REQUIRE(tokens > 0 && H >= 0 && KV >= 0 && H + KV > 0 && Dp > 0 && Dk > 0 && Dk <= Dp, "qkv_prep: bad sizes");
+    RI_REQUIRE(!unit_v || (Dv > 0 && Dv <= Dp), "qkv_prep: values of %d elements in heads of %d", Dv, Dp);
     RI_REQUIRE(Dp <= QP_MAX_DP, "qkv_prep: heads of %d elements exceed the limit %d", Dp, QP_MAX_DP);
     RI_REQUIRE(rot >= 0 && rot <= Dk && rot % 2 == 0, "qkv_prep: %d rotated elements must be even and within the head's %d", rot, Dk);
     RI_REQUIRE(!rope_table || rot > 0, "qkv_prep: a rotation table needs rotated elements");
@@ -378,6 +387,7 @@ extern "C" int ri_qkv_prep_norm(const void* proj, long long ld, int q_col, int k
     a.proj = proj; a.ld = ld; a.q_col = q_col; a.k_col = k_col; a.v_col = v_col; a.bias = bias; a.q_out = q_out;
     a.k_pool = k_pool; a.v_pool = v_pool; a.page_table = page_table; a.tok_seq = tok_seq; a.tok_pos = tok_pos;
     a.seq_slot = seq_slot; a.rope = (const float2*)rope_table; a.rope_rows = rope_rows; a.rot = rope_table ? rot : 0;
+    a.q_factor = q_factor; a.factor_rows = factor_rows; a.unit_v = unit_v; a.Dv = Dv;
     a.q_gain = q_gain; a.k_gain = k_gain; a.norm = norm; a.norm_eps = norm_eps;
     a.pairs = pairs; a.unit = unit; a.eps = eps; a.H = H; a.KV = KV; a.Dp = Dp; a.Dk = Dk; a.mpps = mpps;
     a.page_size = page_size; a.num_pages = num_pages; a.write_kv = write_kv; a.err = err_flag;
@@ -424,14 +434,4 @@ extern "C" int ri_qkv_prep_norm(const void* proj, long long ld, int q_col, int k
     else ri_launch_pdl(qkv_prep_kernel<__nv_bfloat16>, grid, dim3(32 * QP_WARPS), 0, stream, a);
     RI_CHECK_LAUNCH("qkv_prep");
     return 0;
-}
-
-extern "C" int ri_qkv_prep(const void* proj, long long ld, int q_col, int k_col, int v_col, const float* bias, void* q_out,
-                           void* k_pool, void* v_pool, const int* page_table, const int* tok_seq, const int* tok_pos,
-                           const int* seq_slot, const float* rope_table, int rope_rows, int rot, int pairs, int unit,
-                           float eps, int tokens, int H, int KV, int Dp, int Dk, int mpps, int page_size, int num_pages,
-                           int write_kv, int dtype, int* err_flag, cudaStream_t stream) {
-    return ri_qkv_prep_norm(proj, ld, q_col, k_col, v_col, bias, q_out, k_pool, v_pool, page_table, tok_seq, tok_pos, seq_slot,
-                            rope_table, rope_rows, rot, pairs, unit, eps, nullptr, nullptr, 0, 0.0f, tokens, H, KV, Dp, Dk,
-                            mpps, page_size, num_pages, write_kv, dtype, err_flag, stream);
 }

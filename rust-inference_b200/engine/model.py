@@ -81,6 +81,11 @@ class Model:
             self.pass_entry.bind(self.embed_part)
         elif any(e.enters >= 0 for e in spec.schedule):
             raise ValueError("the schedule enters passes, but the model has no pass_entry record")
+        # parts that read the embedding's tables themselves
+        for block in self.blocks:
+            for _, part, _, _ in block.parts():
+                if hasattr(part, "bind"):
+                    part.bind(self.embed_part)
         self.config = None
         self.cache_entry_layers = spec.cache_entries()
         # an embedding that keeps state per sequence has a cache entry of its own, after the layers' entries
@@ -163,7 +168,7 @@ class Model:
         model.config = cfg
         dev = model.env.device
         model.load_tensors(lambda name, info: random_tensor(seed, name, info.shape, info.role, model.env.dtype
-                                                            if info.role == "matrix" else torch.float32, dev))
+                                                            if info.role == "matrix" else torch.float32, dev, below=info.below))
         return model
 
     # ---- what the cache has to hold -----------------------------------------------------------
@@ -202,6 +207,7 @@ class Model:
     # ---- one step ------------------------------------------------------------------------
     def forward(self, ids: torch.Tensor, ctx, cache, want_rows: Optional[torch.Tensor]) -> torch.Tensor:
         """float32 logits [wanted rows, vocab] for the packed tokens ``ids``."""
+        ctx.ids = ids
         with section("embedding"):
             if self.embed_cache_entry is not None:
                 resid = self.embed_part(ids, ctx, cache.layer(self.embed_cache_entry))

@@ -25,9 +25,12 @@ _SIGNATURES = {
     ("elementwise", "ri_embed_rows"): [_P, _P, _P, _I, _I, _I, _I, _P, _P],
     ("elementwise", "ri_embed_rows_scaled"): [_P, _P, _P, _I, _I, _I, _F, _I, _I, _P, _P],
     ("elementwise", "ri_activation"): [_P, _P, _L, _I, _I, _P],
+    ("elementwise", "ri_act_rows"): [_P, _P, _P, _L, _P, _I, _I, _I, _I, _I, _P, _P],
+    ("linear_skinny", "ri_linear_skinny_act_rows"): [_P, _P, _P, _I, _I, _I, _I, _P, _P, _L, _I, _P, _P],
+    ("moe", "ri_moe_plan_table"): [_P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _P, _P],
     ("elementwise", "ri_embed_rows_same"): [_P, _P, _P, _L, _I, _I, _I, _I, _P, _P],
     ("norm_gains", "ri_norm_gains_post"): [_P] * 6 + [_P, _I, _F] + [_P] * 6 + [_I, _I, _F, _P, _F, _L, _I, _P, _I, _I, _P, _P],
-    ("qkv_prep", "ri_qkv_prep_norm"): [_P, _L, _I, _I, _I] + [_P] * 9 + [_I, _I, _I, _I, _F, _P, _P, _I, _F] + [_I] * 10 + [_P, _P],
+    ("qkv_prep", "ri_qkv_prep_norm"): [_P, _L, _I, _I, _I] + [_P] * 9 + [_I, _I, _I, _I, _F, _P, _P, _I, _F, _P, _I, _I, _I] + [_I] * 10 + [_P, _P],
     ("moe", "ri_moe_route_rule"): [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P],
     ("gla", "ri_gla_recurrent_scalar"): [_P, _L, _I, _I, _I, _P, _I, _I, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     ("mlstm", "ri_mlstm_gates"): [_P, _L, _I, _I, _P, _P, _F, _P, _P, _P, _P, _I, _I, _I, _I, _P],
@@ -37,7 +40,7 @@ _SIGNATURES = {
     ("streams", "ri_stream_norm2"): [_P] * 13 + [_I, _I, _I, _F, _I, _I, _P],
     ("pair_embedding", "ri_embed_pair_hash"): [_P] * 9 + [_I, _I, _I, _I, _I, _L, _L, _I, _I, _P, _P],
     ("delta_rule", "ri_short_conv"): [_P, _L, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
-    ("delta_rule", "ri_delta_rule_recurrent"): [_P, _I, _I, _I, _I, _P, _L, _I, _P, _P, _P, _F] + [_P] * 6 + [_I] * 8 + [_P],
+    ("delta_rule", "ri_delta_rule_recurrent"): [_P, _I, _I, _I, _I, _P, _L, _I, _P, _L, _I, _P, _P, _F] + [_P] * 6 + [_I] * 8 + [_P],
     ("elementwise", "ri_gated_act"): [_P, _P, _I, _I, _I, _I, _F, _F, _I, _P],
     ("elementwise", "ri_scale_f32"): [_P, _L, _F, _P],
     ("moe", "ri_moe_route"): [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
@@ -53,25 +56,24 @@ _SIGNATURES = {
     ("elementwise", "ri_add_rows"): [_P, _P, _L, _I, _P],
     ("elementwise", "ri_silu_mul"): [_P, _P, _I, _I, _I, _I, _P],
     ("rope_kv", "ri_qk_norm_rope_append"): [_P] * 10 + [_F, _P, _I, _I] + [_I] * 9 + [_P, _P],
-    ("attention_rows", "ri_attention_rows"): [_P] * 8 + [_I] * 8 + [_F, _I, _P, _F, _I, _P, _P],
+    ("attention_rows", "ri_attention_rows"): [_P] * 8 + [_I] * 8 + [_F, _I, _P, _F, _P, _I, _I, _P, _P],
     ("elementwise", "ri_softcap_f32"): [_P, _L, _F, _P],
     ("norm_gains", "ri_norm_gains"): [_P] * 6 + [_P, _I, _F] + [_P] * 6 + [_I, _I, _F, _I, _P, _I, _I, _P, _P],
-    ("qkv_prep", "ri_qkv_prep"): [_P, _L, _I, _I, _I] + [_P] * 9 + [_I, _I, _I, _I, _F] + [_I] * 10 + [_P, _P],
     ("linear_f32", "ri_linear_f32"): [_P, _P, _P, _I, _I, _I, _P],
     ("sampling", "ri_sample"): [_P, _L, _I, _I, _P, _P, _L, _P, _P, _P, _P, _P, _P, _P, _L, _I, _I, _P, _I, _P],
     ("sampling", "ri_sample_work_bytes"): [_I, _I],
     ("sampling", "ri_argmax"): [_P, _L, _I, _I, _P, _P, _P, _P],
     ("sampling", "ri_mark_seen"): [_P, _L, _P, _P, _I, _I, _P],
     ("attention_decode", "ri_attention_decode_sink"): [_P] * 9 + [_I] * 8 + [_F, _I, _P, _P, _P],
-    ("attention_decode", "ri_attention_decode_cap"): [_P] * 9 + [_I] * 8 + [_F, _I, _P, _F, _P, _P],
+    ("attention_decode", "ri_attention_decode_cap"): [_P] * 9 + [_I] * 8 + [_F, _I, _P, _F, _P, _I, _P, _P],
     ("linear_skinny", "ri_linear_skinny"): [_P, _P, _P, _I, _I, _I, _I, _I, _P, _P],
     ("linear_skinny", "ri_linear_skinny_act"): [_P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P],
     ("linear_skinny", "ri_linear_skinny_gated"): [_P, _P, _P, _I, _I, _I, _I, _P, _P],
     ("linear_skinny", "ri_linear_skinny_gated_with"): [_P, _P, _P, _I, _I, _I, _I, _F, _F, _P, _P],
     ("linear_stream_tc", "ri_linear_stream_tc"): [_P, _P, _P, _I, _I, _I, _I, _I, _P, _P],
     ("linear_stream_tc", "ri_linear_stream_tc_gate"): [_P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P, _P],
-    ("attention_prefill_tc", "ri_attention_prefill_tc"): [_P] * 8 + [_I] * 9 + [_F, _I, _P, _F, _P, _P],
-    ("attention_prefill", "ri_attention_prefill"): [_P] * 8 + [_I] * 8 + [_F, _I, _P, _I, _F, _P, _P],
+    ("attention_prefill_tc", "ri_attention_prefill_tc"): [_P] * 8 + [_I] * 9 + [_F, _I, _P, _F, _P, _I, _P, _P],
+    ("attention_prefill", "ri_attention_prefill"): [_P] * 8 + [_I] * 8 + [_F, _I, _P, _I, _F, _P, _I, _P, _P],
 }
 DECODE_CHUNK = 128          # keys per partial result of the decode attention kernel
 MAX_FAST_HEAD_DIM = 256
@@ -213,7 +215,8 @@ ERROR_TEXT = {1: "token id outside the vocabulary", 2: "cache write to an unmapp
               6: "the tcgen05 attention kernel's shared memory does not start on a multiple of 1024 bytes "
                  "(set RUST_INFERENCE_B200_NO_TCGEN05=1 to use the mma.sync kernel)",
               7: "a sequence is longer than the scratch memory given to the decode attention covers "
-                 "(max_chunks x 128 keys): the keys beyond were left out"}
+                 "(max_chunks x 128 keys): the keys beyond were left out",
+              8: "a table of experts names an expert that does not exist"}
 
 
 # ---------------------------------------------------------------------------------------
@@ -634,6 +637,33 @@ def linear_act(x: torch.Tensor, w: torch.Tensor, act: str) -> torch.Tensor:
     return activation(linear(x, w), act)
 
 
+def linear_act_rows(x: torch.Tensor, w: torch.Tensor, act: str, ids: torch.Tensor, rows: torch.Tensor) -> torch.Tensor:
+    """act(x w^T)[t] * rows[ids[t]] for x [M, K], w [N, K], ``rows`` [vocab, N] (it may be a block of columns of a wider
+    table) and int32 ``ids`` [M].  A handful of bfloat16 tokens run as one kernel (the weight-streaming product's
+    epilogue); otherwise the product is followed by ``act_rows``."""
+    if act not in ACTIVATIONS:
+        raise KernelError(f"activation {act!r} is not built (known: {', '.join(sorted(ACTIVATIONS))})")
+    M, K = x.shape
+    N = w.shape[0]
+    _need(ids, "ids", torch.int32, (M,))
+    ld = _columns(rows, "rows", x.dtype)
+    if rows.shape[1] != N:
+        raise KernelError(f"linear_act_rows: rows {tuple(rows.shape)} do not fit {N} outputs")
+    if x.dtype == torch.bfloat16 and w.shape[1] == K and _FUSED_ACT and _takes_skinny(M, N, K, x.device):
+        _need(x, "x")
+        _need(w, "w", x.dtype)
+        y = torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
+        _call("linear_skinny", "ri_linear_skinny_act_rows", x.data_ptr(), w.data_ptr(), y.data_ptr(), M, N, K,
+              ACTIVATIONS[act] + 1, ids.data_ptr(), rows.data_ptr(), int(ld), rows.shape[0], error_flag(x.device).data_ptr(),
+              _stream())
+        return y
+    z = linear(x, w)
+    out = torch.empty_like(z)
+    _call("elementwise", "ri_act_rows", z.data_ptr(), ids.data_ptr(), rows.data_ptr(), int(ld), out.data_ptr(), M, N,
+          rows.shape[0], ACTIVATIONS[act], _code(z.dtype), error_flag(z.device).data_ptr(), _stream())
+    return out
+
+
 def linear(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     """y = x w^T for x [M, K], w [N, K].
 
@@ -761,7 +791,7 @@ def rms_gains(resid: torch.Tensor, gains, eps: float, out_dtype: torch.dtype, te
     _need(resid, "resid", torch.float32)
     n, dim = resid.shape
     gains = tuple(gains)
-    if len(gains) > 2 or (not gains and (rows is not None or then is not None)):
+    if len(gains) > 2 or (not gains and rows is not None):
         raise KernelError(f"rms_gains: {len(gains)} gains (one or two; none only for whole steps)")
     for g in gains:
         _need(g, "gain", torch.float32, (dim,))
@@ -831,7 +861,8 @@ def qkv_prep(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, heads: int,
              eps: float, k_pool: Optional[torch.Tensor], v_pool: Optional[torch.Tensor], page_table: torch.Tensor,
              tok_seq: torch.Tensor, tok_pos: torch.Tensor, seq_slot: torch.Tensor, write_kv: bool = True,
              norm: str = "", q_gain: Optional[torch.Tensor] = None, k_gain: Optional[torch.Tensor] = None,
-             norm_eps: float = 0.0) -> torch.Tensor:
+             norm_eps: float = 0.0, q_factor: Optional[torch.Tensor] = None, unit_v: bool = False,
+             Dv: int = 0) -> torch.Tensor:
     """Between the q/k/v product and the attention kernels: ``proj`` [tokens, N] holds the q heads from column ``q_col``,
     the k heads from ``k_col`` and the v heads from ``v_col`` (< 0: none, the values are the keys as cached), every head
     ``Dp`` columns wide with ``Dk`` true elements.  ``bias`` (float32, by column of the product) is added first; the first
@@ -842,14 +873,18 @@ def qkv_prep(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, heads: int,
 
     ``norm``: an RMS norm of q and k before the rotation, "head" over each head's ``Dk`` elements with the gains
     ``q_gain`` and ``k_gain`` [Dp] for all heads, or "all" over all q heads (all k heads) of the token at once with gains
-    [H, Dp] and [KV, Dp]; eps ``norm_eps`` inside the root; the gains' padding columns are zero."""
+    [H, Dp] and [KV, Dp]; eps ``norm_eps`` inside the root; the gains' padding columns are zero.
+
+    ``q_factor`` [positions] (float32): the finished q heads are multiplied by their position's entry.  ``unit_v``: v heads
+    are divided by their root mean square over ``Dv`` elements (eps ``eps``).  ``kv_heads`` 0: only queries."""
     _need(proj, "proj")
     tokens, ld = proj.shape
     if norm not in ("", "head", "all"):
         raise KernelError(f"qkv_prep: norm {norm!r} (head, all or none)")
     if norm:
         for g, name, n in ((q_gain, "q_gain", heads), (k_gain, "k_gain", kv_heads)):
-            _need(g, name, torch.float32, (Dp,) if norm == "head" else (n, Dp))
+            if n:
+                _need(g, name, torch.float32, (Dp,) if norm == "head" else (n, Dp))
     nv = 0 if v_col < 0 else kv_heads
     if q_col + heads * Dp > ld or k_col + kv_heads * Dp > ld or (nv and v_col + nv * Dp > ld):
         raise KernelError("qkv_prep: the projection is narrower than its columns")
@@ -858,6 +893,8 @@ def qkv_prep(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, heads: int,
         if bias.numel() < max(q_col + heads * Dp, k_col + kv_heads * Dp, v_col + nv * Dp):
             raise KernelError("qkv_prep: the bias vector is shorter than the columns it is indexed by")
     rope_rows = 0
+    if q_factor is not None:
+        _need(q_factor, "q_factor", torch.float32)
     if rope_table is not None:
         _need(rope_table, "rope_table", torch.float32)
         if rope_table.dim() != 3 or rope_table.shape[1] != rot // 2 or rope_table.shape[2] != 2:
@@ -882,7 +919,8 @@ def qkv_prep(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, heads: int,
           _ptr(k_pool) if write_kv else None, _ptr(v_pool) if write_kv and nv else None, page_table.data_ptr(),
           tok_seq.data_ptr(), tok_pos.data_ptr(), seq_slot.data_ptr(), _ptr(rope_table), rope_rows, int(rot),
           1 if pairs else 0, 1 if unit else 0, float(eps), _ptr(q_gain) if norm else None, _ptr(k_gain) if norm else None,
-          {"": 0, "head": 1, "all": 2}[norm], float(norm_eps), tokens, heads, kv_heads, Dp, Dk, page_table.shape[1], page_size,
+          {"": 0, "head": 1, "all": 2}[norm], float(norm_eps), _ptr(q_factor), 0 if q_factor is None else q_factor.numel(),
+          1 if unit_v else 0, int(Dv or Dk), tokens, heads, kv_heads, Dp, Dk, page_table.shape[1], page_size,
           pages, 1 if write_kv else 0, _code(proj.dtype), error_flag(proj.device).data_ptr(), _stream())
     return q
 
@@ -909,15 +947,27 @@ def _sink(sink: Optional[torch.Tensor], heads: int) -> Optional[int]:
     return sink.data_ptr()
 
 
+def _bias(dist_bias: Optional[torch.Tensor], heads: int):
+    """(pointer, entries per head) of a distance bias [heads, n], (None, 0) for none."""
+    if dist_bias is None:
+        return None, 0
+    _need(dist_bias, "dist_bias", torch.float32)
+    if dist_bias.dim() != 2 or dist_bias.shape[0] != heads or dist_bias.shape[1] < 1:
+        raise KernelError(f"attention: distance bias {tuple(dist_bias.shape)} does not fit {heads} heads")
+    return dist_bias.data_ptr(), dist_bias.shape[1]
+
+
 def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_table: torch.Tensor,
               seq_slot: torch.Tensor, seq_start: torch.Tensor, seq_len: torch.Tensor, max_new: int, scale: float,
-              window: int = 0, sink: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0) -> torch.Tensor:
+              window: int = 0, sink: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0,
+              dist_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of the step's new tokens (q [tokens, H, Dh], sequences back to back as
     ``seq_start`` says) over the paged cache, which already holds their keys and values: float32 or
     bfloat16, any head size up to 512, any page size.  Every (token, head) is computed in one fixed
     order that depends on its own position only, so the result does not depend on the step's cutting.
     ``sink`` [H] (float32): exp(sink[h]) joins head h's softmax denominator, with no key and no value.
     ``softcap`` > 0: score <- softcap * tanh(score / softcap) after the scale.
+    ``dist_bias`` [H, n] (float32): added to the score after that, entry min(distance, n - 1) of the head's row.
     ``v_pool`` may be ``k_pool`` itself (values that are the keys: latent attention)."""
     _need(q, "q")
     tokens, H, Dh = q.shape
@@ -935,7 +985,7 @@ def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_
     _call("attention_rows", "ri_attention_rows", q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), out.data_ptr(),
           page_table.data_ptr(), seq_slot.data_ptr(), seq_start.data_ptr(), seq_len.data_ptr(), seqs, int(max_new),
           H, KV, Dh, page_table.shape[1], page_size, pages, float(scale), _mask(window, chunk), _sink(sink, H), _cap(softcap),
-          _code(q.dtype), error_flag(q.device).data_ptr(), _stream())
+          *_bias(dist_bias, H), _code(q.dtype), error_flag(q.device).data_ptr(), _stream())
     return out
 
 
@@ -952,7 +1002,8 @@ def _decode_parts(head_dim: int, chunks: int) -> int:
 
 def attention_decode(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_table: torch.Tensor,
                      seq_slot: torch.Tensor, seq_len: torch.Tensor, scale: float, window: int,
-                     max_len: int, sink: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0) -> torch.Tensor:
+                     max_len: int, sink: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0,
+                     dist_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of one new token per sequence (q [seqs, H, Dh], bfloat16) over the
     paged cache, keys split into chunks of ``DECODE_CHUNK``; ``max_len`` bounds the
     sequences' lengths after this step and sizes the scratch memory."""
@@ -976,7 +1027,7 @@ def attention_decode(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
     _call("attention_decode", "ri_attention_decode_cap", q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(),
           out.data_ptr(), o_part.data_ptr(), ml_part.data_ptr(), page_table.data_ptr(), seq_slot.data_ptr(),
           seq_len.data_ptr(), seqs, H, KV, Dh, page_table.shape[1], page_size, pages, chunks, float(scale),
-          _mask(window, chunk), _sink(sink, H), _cap(softcap), error_flag(q.device).data_ptr(), _stream(),
+          _mask(window, chunk), _sink(sink, H), _cap(softcap), *_bias(dist_bias, H), error_flag(q.device).data_ptr(), _stream(),
           defines={"RI_HEAD_DIM": Dh})
     return out
 
@@ -984,7 +1035,7 @@ def attention_decode(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
 def attention_prefill(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_table: torch.Tensor,
                       seq_slot: torch.Tensor, seq_start: torch.Tensor, seq_len: torch.Tensor, max_new: int,
                       scale: float, window: int, sink: Optional[torch.Tensor] = None, v_dims: int = 0,
-                      chunk: int = 0, softcap: float = 0.0) -> torch.Tensor:
+                      chunk: int = 0, softcap: float = 0.0, dist_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of the step's new tokens (q [tokens, H, Dh], bfloat16, sequences back
     to back as ``seq_start`` says) over the paged cache, which already holds their keys
     and values; ``max_new`` is the most tokens one sequence brings.  ``v_pool`` may be ``k_pool``
@@ -1010,13 +1061,13 @@ def attention_prefill(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tenso
         _call("attention_prefill_tc", "ri_attention_prefill_tc", q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(),
               out.data_ptr(), page_table.data_ptr(), seq_slot.data_ptr(), seq_start.data_ptr(), seq_len.data_ptr(),
               q.shape[0], seqs, int(max_new), H, KV, Dh, page_table.shape[1], page_size, pages, float(scale),
-              _mask(window, chunk), _sink(sink, H), _cap(softcap), error_flag(q.device).data_ptr(), _stream(),
+              _mask(window, chunk), _sink(sink, H), _cap(softcap), *_bias(dist_bias, H), error_flag(q.device).data_ptr(), _stream(),
               defines={"RI_HEAD_DIM": Dh})
         return out
     _call("attention_prefill", "ri_attention_prefill", q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(),
           out.data_ptr(), page_table.data_ptr(), seq_slot.data_ptr(), seq_start.data_ptr(), seq_len.data_ptr(),
           seqs, int(max_new), H, KV, Dh, page_table.shape[1], page_size, pages, float(scale), _mask(window, chunk),
-          _sink(sink, H), int(v_dims), _cap(softcap), error_flag(q.device).data_ptr(), _stream(), defines={"RI_HEAD_DIM": Dh})
+          _sink(sink, H), int(v_dims), _cap(softcap), *_bias(dist_bias, H), error_flag(q.device).data_ptr(), _stream(), defines={"RI_HEAD_DIM": Dh})
     return out
 
 
@@ -1173,13 +1224,17 @@ def delta_rule_recurrent(qkv: torch.Tensor, q_col: int, k_col: int, v_col: int, 
     S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q, with q and k made unit vectors (q also times
     ``qscale``), g = exp(-exp(a_log[h]) softplus(z + dt_bias)) per key channel and beta = sigmoid of column
     ``beta_col + h`` of ``proj``.  ``qkv`` [tokens, C] float32 holds q, k, v from ``q_col``, ``k_col``, ``v_col``;
-    ``z`` [tokens, H*dim] in the compute dtype.  The q and k columns of ``qkv`` are made unit vectors in place.
+    ``z`` [tokens, H*dim] in the compute dtype (or [tokens, H] with ``dt_bias`` [H]: one decay per head for all its
+    channels; it may be a block of columns of a wider matrix).  The q and k columns of ``qkv`` are made unit vectors in place.
     Returns o [tokens, H, vdim] float32."""
     _need(qkv, "qkv", torch.float32)
     tokens, C = qkv.shape
     _need(proj, "proj")
-    _need(z, "z", proj.dtype, (tokens, heads * dim))
-    _need(dt_bias, "dt_bias", torch.float32, (heads * dim,))
+    ddim = dim if z.shape[1] == heads * dim else 1
+    ldz = _columns(z, "z", proj.dtype)
+    if tuple(z.shape) != (tokens, heads * ddim):
+        raise KernelError(f"delta_rule_recurrent: decays {tuple(z.shape)} do not fit {tokens} tokens of {heads} heads")
+    _need(dt_bias, "dt_bias", torch.float32, (heads * ddim,))
     _need(a_log, "a_log", torch.float32, (heads,))
     _need(state, "state", torch.float32)
     if tuple(state.shape[1:]) != (heads, dim, vdim):
@@ -1190,10 +1245,10 @@ def delta_rule_recurrent(qkv: torch.Tensor, q_col: int, k_col: int, v_col: int, 
     _need(seq_slot, "seq_slot", torch.int32, (seqs,))
     _need(seq_start, "seq_start", torch.int32, (seqs + 1,))
     o = torch.empty((tokens, heads, vdim), dtype=torch.float32, device=qkv.device)
-    decay = torch.empty((tokens, heads * dim), dtype=torch.float32, device=qkv.device)
+    decay = torch.empty((tokens, heads * ddim), dtype=torch.float32, device=qkv.device)
     beta = torch.empty((tokens, heads + qk_heads), dtype=torch.float32, device=qkv.device)
     _call("delta_rule", "ri_delta_rule_recurrent", qkv.data_ptr(), C, int(q_col), int(k_col), int(v_col), proj.data_ptr(),
-          proj.shape[1], int(beta_col), z.data_ptr(), dt_bias.data_ptr(), a_log.data_ptr(), float(qscale), decay.data_ptr(),
+          proj.shape[1], int(beta_col), z.data_ptr(), int(ldz), ddim, dt_bias.data_ptr(), a_log.data_ptr(), float(qscale), decay.data_ptr(),
           beta.data_ptr(), state.data_ptr(), o.data_ptr(), seq_slot.data_ptr(), seq_start.data_ptr(), tokens, seqs, heads,
           qk_heads, dim, vdim, 1 if single and tokens == seqs else 0, _code(proj.dtype), _stream())
     add_launches(1)
@@ -1303,6 +1358,25 @@ def moe_plan(idx: torch.Tensor, experts: int, wide: bool = False):
     return perm, tiles, meta, bm
 
 
+def moe_plan_table(ids: torch.Tensor, table: torch.Tensor, experts: int, wide: bool = False):
+    """The plan of a step whose experts an integer table [vocab, top] names by token id (no router): (idx int32 [tokens,
+    top] = table[ids], plan as ``moe_plan`` gives it), in one launch."""
+    _need(ids, "ids", torch.int32)
+    _need(table, "table", torch.int32)
+    tokens, (vocab, top) = ids.numel(), table.shape
+    pairs = tokens * top
+    bm = MOE_TILE_ROWS_WIDE if wide else MOE_TILE_ROWS
+    _, lib = _fn("moe", "ri_moe_plan_table")
+    max_tiles = int(lib.ri_moe_max_tiles(int(pairs), int(experts), bm))
+    idx = torch.empty((tokens, top), dtype=torch.int32, device=ids.device)
+    perm = torch.empty(max(pairs, 1), dtype=torch.int32, device=ids.device)
+    tiles = torch.empty((max_tiles, 3), dtype=torch.int32, device=ids.device)
+    meta = torch.empty(2, dtype=torch.int32, device=ids.device)
+    _call("moe", "ri_moe_plan_table", ids.data_ptr(), table.data_ptr(), vocab, top, idx.data_ptr(), perm.data_ptr(),
+          tiles.data_ptr(), meta.data_ptr(), tokens, int(experts), max_tiles, bm, error_flag(ids.device).data_ptr(), _stream())
+    return idx, (perm, tiles, meta, bm)
+
+
 def moe_grouped_linear(a: torch.Tensor, w: torch.Tensor, plan, rows_out: int, gather_div: int = 0, scatter: bool = False,
                        out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     """y[out(r)] = w[e] a[in(r)] for every row r of the plan's tiles; ``w`` [E, N, K]; in(r) = perm[r] // gather_div
@@ -1323,19 +1397,20 @@ def moe_grouped_linear(a: torch.Tensor, w: torch.Tensor, plan, rows_out: int, ga
     return y
 
 
-def moe_combine(pair_out: torch.Tensor, idx: torch.Tensor, weight: torch.Tensor, x: torch.Tensor, experts: int,
+def moe_combine(pair_out: torch.Tensor, idx: torch.Tensor, weight: Optional[torch.Tensor], x: torch.Tensor, experts: int,
                 extra: Optional[torch.Tensor] = None) -> torch.Tensor:
     """y[t] = sum_j weight[t, j] * (idx[t, j] >= experts ? x[t] : pair_out[t * top + j]) (+ extra[t]), in float32, j
-    ascending, rounded once to x's dtype."""
+    ascending, rounded once to x's dtype.  ``weight`` None: every choice weighs 1 / top."""
     _need(x, "x")
     tokens, D = x.shape
     top = idx.shape[1]
     _need(pair_out, "pair_out", torch.float32, (tokens * top, D))
     _need(idx, "idx", torch.int32, (tokens, top))
-    _need(weight, "weight", torch.float32, (tokens, top))
+    if weight is not None:
+        _need(weight, "weight", torch.float32, (tokens, top))
     if extra is not None:
         _need(extra, "extra", x.dtype, (tokens, D))
     y = torch.empty_like(x)
-    _call("moe", "ri_moe_combine", pair_out.data_ptr(), idx.data_ptr(), weight.data_ptr(), x.data_ptr(), _ptr(extra),
+    _call("moe", "ri_moe_combine", pair_out.data_ptr(), idx.data_ptr(), _ptr(weight), x.data_ptr(), _ptr(extra),
           y.data_ptr(), tokens, D, top, int(experts), _code(x.dtype), _stream())
     return y

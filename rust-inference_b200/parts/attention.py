@@ -18,7 +18,10 @@ Further options of the record, each a field with its constants: biases on the q/
 (no v tensor, one pool), queries and keys divided by their root mean square AFTER the rotation
 (no gain), a soft-cap on the scores, and a sigmoid gate per output element from a projection of
 the mixer's input (or one gate per head), stacked into the q/k/v product; a norm of queries and keys
-before the rotation that runs over the whole projection of a token instead of over each head.  A record
+before the rotation that runs over the whole projection of a token instead of over each head; values divided by
+their root mean square before they are cached; a factor on the queries that grows with the position; a learned
+bias on the scores by distance (``parts/distance.py``); no keys and values of its own (the layer reads the cache
+entry that another layer writes).  A record
 that uses any of them (or a per-head norm together with values of another size) runs the
 "extended" order of work: one product for q, k, (v), (gate); ``ops.qkv_prep`` (bias, rotation,
 unit norm, append); attention; gate; output projection.  Heads are then always padded to a
@@ -33,6 +36,7 @@ import torch
 from .. import ops
 from ..profiler import section
 from .base import CacheRequest, Mixer, PositionEncoding
+from .distance import spread_over_distances
 from .registry import ParamInfo, build_part, register_mixer
 
 
@@ -70,13 +74,21 @@ class Attention(Mixer):
             raise ValueError(f"gate {self.gated!r} is not built (known: element, head)")
         if set(self.bias_of) - {"q", "k", "v"}:
             raise ValueError(f"biases {self.bias_of}: of q, k, v")
+        self.unit_values = bool(getattr(spec, "unit_values", False))
+        self.temperature = getattr(spec, "temperature", None)
+        self.bias_rows = int(getattr(spec, "bias_rows", 0) or 0)
+        self.own_kv = bool(getattr(spec, "own_kv", True))
+        self.q_factor = self.dist_bias = None
         self.extended = bool(self.bias_of or self.keys_are_values or self.unit_rms or self.softcap or self.gated
+                             or self.unit_values or self.temperature or self.bias_rows or not self.own_kv
                              or self.norm_span == "all" or (self.norm_span and self.Dp != self.Dk))
         if self.extended:
             if spec.sink or spec.chunk:
                 raise ValueError("the extended attention options do not combine with a sink or a chunked mask")
             if self.keys_are_values and self.Dv != self.Dk:
                 raise ValueError(f"values that are the keys have the keys' size {self.Dk}, not {self.Dv}")
+            if self.unit_values and self.keys_are_values:
+                raise ValueError("values that are the keys are cached as the keys are, without a norm of their own")
             self.Dp = -(-max(self.Dk, self.Dv) // 16) * 16
             self.bias = None
 
@@ -86,8 +98,12 @@ class Attention(Mixer):
         Dv = spec.v_head_dim or Dh
         q, k, v, o, sink = spec.names
         infos = {q: ParamInfo((H * Dh, D)), k: ParamInfo((KV * Dh, D)), v: ParamInfo((KV * Dv, D)), o: ParamInfo((D, H * Dv))}
-        if getattr(spec, "values", "own") == "keys":
+        if getattr(spec, "values", "own") == "keys" or not getattr(spec, "own_kv", True):
             del infos[v]
+        if not getattr(spec, "own_kv", True):
+            del infos[k]
+        if getattr(spec, "bias_rows", 0):
+            infos[spec.bias_name] = ParamInfo((spec.bias_rows, H), "vector")
         suffix = getattr(spec, "bias_suffix", ".b")
         for which, name in (("q", q), ("k", k), ("v", v)):
             if which in (getattr(spec, "bias", ()) or ()) and name in infos:
@@ -98,7 +114,8 @@ class Attention(Mixer):
             qn, kn = getattr(spec, "qk_norm_names", ("q_norm.weight", "k_norm.weight"))
             whole = getattr(spec, "qk_norm_span", "head") == "all"
             infos[qn] = ParamInfo((H * Dh if whole else Dh,), "gain")
-            infos[kn] = ParamInfo((KV * Dh if whole else Dh,), "gain")
+            if getattr(spec, "own_kv", True):
+                infos[kn] = ParamInfo((KV * Dh if whole else Dh,), "gain")
         if spec.sink:
             infos[sink] = ParamInfo((H,), "vector")
         return infos
@@ -115,8 +132,11 @@ class Attention(Mixer):
             out[:, :size] = t.view(heads, size, D)
             return out.view(heads * Dp, D)
 
-        blocks = [rows(tensors[q], s.num_heads, self.Dk), rows(tensors[k], s.num_kv_heads, self.Dk)]
-        if not self.keys_are_values:
+        own = self.own_kv
+        blocks = [rows(tensors[q], s.num_heads, self.Dk)]
+        if own:
+            blocks.append(rows(tensors[k], s.num_kv_heads, self.Dk))
+        if own and not self.keys_are_values:
             blocks.append(rows(tensors[v], s.num_kv_heads, self.Dv))
         if self.gated == "element":
             blocks.append(rows(tensors[s.gate_name], s.num_heads, self.Dv))
@@ -130,16 +150,16 @@ class Attention(Mixer):
         if self.extended:
             # the columns of the product: q heads, k heads, v heads (unless the keys serve), gate; the biases as one
             # float32 vector over the q/k/v columns, zero where a projection has none and in the padding
-            H, KV = s.num_heads, s.num_kv_heads
-            self.k_col = H * Dp
-            self.v_col = -1 if self.keys_are_values else (H + KV) * Dp
+            H, KV = s.num_heads, s.num_kv_heads if own else 0
+            self.k_col = H * Dp if own else 0
+            self.v_col = -1 if self.keys_are_values or not own else (H + KV) * Dp
             self.g_col = (H + KV + (0 if self.keys_are_values else KV)) * Dp
             self.bias = None
             if self.bias_of:
                 bias = torch.zeros(self.g_col, dtype=torch.float32, device=self.qkv.device)
                 for which, name, col, heads, size in (("q", q, 0, H, self.Dk), ("k", k, self.k_col, KV, self.Dk),
                                                       ("v", v, self.v_col, KV, self.Dv)):
-                    if which in self.bias_of and col >= 0:
+                    if which in self.bias_of and col >= 0 and heads:
                         bias[col:col + heads * Dp].view(heads, Dp)[:, :size] = tensors[name + s.bias_suffix].float().view(heads, size)
                 self.bias = bias
         wo = tensors[o]
@@ -150,7 +170,7 @@ class Attention(Mixer):
         self.o = wo.contiguous()
         if s.qk_norm is not None:
             qn, kn = getattr(s, "qk_norm_names", ("q_norm.weight", "k_norm.weight"))
-            self.q_gain, self.k_gain = tensors[qn], tensors[kn]
+            self.q_gain, self.k_gain = tensors[qn], tensors.get(kn)
             if self.extended:
                 # the kernel indexes the gains by the padded head's column: zeros in the padding
                 def padded(g, heads):
@@ -161,9 +181,12 @@ class Attention(Mixer):
                         out = g.new_zeros((heads, Dp))
                         out[:, :self.Dk] = g.view(heads, self.Dk)
                     return out.contiguous()
-                self.q_gain, self.k_gain = padded(self.q_gain, s.num_heads), padded(self.k_gain, s.num_kv_heads)
+                self.q_gain = padded(self.q_gain, s.num_heads)
+                self.k_gain = padded(self.k_gain, s.num_kv_heads) if own else None
         if s.sink:
             self.sink = tensors[sink]
+        if self.bias_rows:
+            self.dist_bias = spread_over_distances(tensors[s.bias_name], s.bias_far)
 
     def weight_bytes(self):
         return (self.qkv.numel() + self.o.numel()) * self.qkv.element_size()
@@ -178,10 +201,17 @@ class Attention(Mixer):
 
     def prepare(self, max_positions):
         self.position.prepare(max_positions)
+        if self.temperature and (self.q_factor is None or self.q_factor.numel() < max_positions):
+            coef, every = self.temperature
+            p = torch.arange(max_positions, dtype=torch.float64)
+            f = 1.0 + coef * torch.log(torch.floor((p + 1.0) / every) + 1.0)
+            self.q_factor = f.to(device=self.env.device, dtype=torch.float32)
 
     def _extended(self, x, ctx, cache):
         s = self.spec
-        T, H, KV, Dp = x.shape[0], s.num_heads, s.num_kv_heads, self.Dp
+        T, H, KV, Dp = x.shape[0], s.num_heads, s.num_kv_heads if self.own_kv else 0, self.Dp
+        if cache.writes and not self.own_kv:
+            raise ValueError("a layer without keys and values of its own reads a cache entry and cannot write it")
         with section("attn q/k/v proj"):
             proj = ops.linear(x, self.qkv)
         table = self.position.fused_table()
@@ -192,19 +222,22 @@ class Attention(Mixer):
                              self.rot if table is not None else 0, getattr(self.position, "pairs", False),
                              self.unit_rms, s.unit_eps, cache.k_pool, cache.v_pool, cache.page_table, ctx.tok_seq,
                              ctx.tok_pos, ctx.seq_slot, write_kv=cache.writes, norm=self.norm_span, q_gain=self.q_gain,
-                             k_gain=self.k_gain, norm_eps=s.qk_norm.eps if s.qk_norm is not None else 0.0)
+                             k_gain=self.k_gain, norm_eps=s.qk_norm.eps if s.qk_norm is not None else 0.0,
+                             q_factor=self.q_factor, unit_v=self.unit_values, Dv=self.Dv)
         fast = ops.fast_attention_supported(q.dtype, Dp, cache.page_size)
         with section("attention"):
             if fast and ctx.decode_only:
                 out = ops.attention_decode(q, cache.k_pool, cache.v_pool, cache.page_table, ctx.seq_slot, ctx.seq_len,
-                                           self.scale, s.window, ctx.len_bucket, softcap=self.softcap)
+                                           self.scale, s.window, ctx.len_bucket, softcap=self.softcap,
+                                           dist_bias=self.dist_bias)
             elif fast:
                 out = ops.attention_prefill(q, cache.k_pool, cache.v_pool, cache.page_table, ctx.seq_slot,
                                             ctx.seq_start, ctx.seq_len, ctx.max_new, self.scale, s.window,
-                                            softcap=self.softcap)
+                                            softcap=self.softcap, dist_bias=self.dist_bias)
             else:
                 out = ops.attention(q, cache.k_pool, cache.v_pool, cache.page_table, ctx.seq_slot, ctx.seq_start,
-                                    ctx.seq_len, ctx.max_new, self.scale, s.window, softcap=self.softcap)
+                                    ctx.seq_len, ctx.max_new, self.scale, s.window, softcap=self.softcap,
+                                    dist_bias=self.dist_bias)
         if self.gated:
             with section("attn gate"):
                 ops.gate_heads(out, proj[:, self.g_col:self.g_col + (H if self.gated == "head" else H * Dp)], "sigmoid")

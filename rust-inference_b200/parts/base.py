@@ -47,6 +47,7 @@ class StepContext:
     seq_slot[b]  cache slot of sequence b
     seq_start[b] first packed token of sequence b (length B+1)
     seq_len[b]   length of sequence b after this step
+    ids[t]       token id of token t (for parts that look something up by it; the model sets it)
     """
     tok_seq: torch.Tensor
     tok_pos: torch.Tensor
@@ -60,6 +61,7 @@ class StepContext:
     host_seq_slot: tuple = ()
     host_new: tuple = ()          # tokens each sequence brings
     host_len: tuple = ()          # lengths after this step
+    ids: Optional[torch.Tensor] = None
 
     @property
     def decode_only(self) -> bool:

@@ -143,6 +143,33 @@ class SandwichBlock(BlockBase):
         return resid, self.ffn_link.pending(self.ffn(x, ctx))
 
 
+@register_block("postnorm")
+class PostNormBlock(BlockBase):
+    """Sublayers that read the residual itself, each with a norm behind it: x <- x + link1(mixer(x)),
+    x <- x + link2(ffn(x)), x <- x + link3(side(x)); the feed-forward and the token-fed sublayer are optional.  As in the
+    other arrangements an output is left pending: the reader in front of the next sublayer norms it, adds it and hands
+    over the new residual in one pass."""
+
+    @classmethod
+    def slots(cls, spec):
+        out = [("reader", "norm", spec.reader), ("mixer_link", "link", spec.mixer_link), ("mixer", "mixer", spec.mixer)]
+        for name in ("ffn", "side"):
+            if getattr(spec, name) is not None:
+                out += [(name + "_link", "link", getattr(spec, name + "_link")), (name, "ffn", getattr(spec, name))]
+        return tuple(out)
+
+    def __call__(self, resid, delta, ctx, cache):
+        x = norm_before(self.reader, resid, delta, self.mixer)
+        delta = self.mixer_link.pending(self.mixer(x, ctx, cache))
+        if self.spec.ffn is not None:
+            x = norm_before(self.reader, resid, delta, self.ffn)
+            delta = self.ffn_link.pending(self.ffn(x, ctx))
+        if self.spec.side is not None:
+            x = norm_before(self.reader, resid, delta, self.side)
+            delta = self.side_link.pending(self.side(x, ctx))
+        return resid, delta
+
+
 def norm_before(norm, resid, delta, reader):
     """``norm(resid + delta)`` for the part ``reader``; a norm that takes hints is told which matrix is read next."""
     if norm.takes_hint:

@@ -33,10 +33,15 @@ class TokenEmbedding(Part):
 
     @classmethod
     def param_infos(cls, spec):
-        return {"weight": ParamInfo((spec.vocab_size, spec.hidden_size), "matrix")}
+        infos = {"weight": ParamInfo((spec.vocab_size, spec.hidden_size), "matrix")}
+        if getattr(spec, "side_width", 0):
+            infos[spec.side_name] = ParamInfo((spec.vocab_size, spec.side_width), "matrix")
+        return infos
 
     def load(self, tensors):
         self.table = tensors["weight"]
+        # a second table of token rows: the layers' token-fed sublayers read their columns of it
+        self.side = tensors[self.spec.side_name] if getattr(self.spec, "side_width", 0) else None
 
     def weight_bytes(self):
         return self.table.numel() * self.table.element_size()

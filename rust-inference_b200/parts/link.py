@@ -95,7 +95,8 @@ class PostNormLink(Part):
 
     @classmethod
     def param_infos(cls, spec):
-        infos = {spec.gain_name: ParamInfo((spec.size,), "vector" if spec.one_plus else "gain")}
+        shape = () if getattr(spec, "scalar", False) else (spec.size,)
+        infos = {spec.gain_name: ParamInfo(shape, "vector" if spec.one_plus else "gain")}
         if spec.scale_name:
             infos[spec.scale_name] = ParamInfo((spec.size,), "gain")
         return infos
@@ -104,6 +105,8 @@ class PostNormLink(Part):
         g = tensors[self.spec.gain_name]
         if self.spec.one_plus:
             g = g + 1.0
+        if getattr(self.spec, "scalar", False):
+            g = g.reshape(1).expand(self.spec.size)
         if self.spec.scale_name:
             g = g * tensors[self.spec.scale_name]
         self.gain = g.contiguous()

@@ -85,6 +85,46 @@ class GatedFF(FeedForward):
             return ops.linear(z, self.down)
 
 
+@register_ffn("token_side")
+class TokenSide(FeedForward):
+    """proj(gelu_tanh(gate x) * e) with e this layer's columns of the token's row in the embedding's second table (a table
+    that all layers share).  For a handful of tokens the gate's product applies the activation and the row itself."""
+    graph_safe = True
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.embedding = None
+
+    @classmethod
+    def param_infos(cls, spec):
+        D, E = spec.hidden_size, spec.size
+        return {"gate": ParamInfo((E, D)), "proj": ParamInfo((D, E))}
+
+    def load(self, tensors):
+        self.gate, self.proj = tensors["gate"].contiguous(), tensors["proj"].contiguous()
+
+    def bind(self, embedding) -> None:
+        """The model's embedding part, whose ``side`` table holds the rows."""
+        s = self.spec
+        width = getattr(embedding.spec, "side_width", 0)
+        if s.start < 0 or s.start + s.size > width:
+            raise ValueError(f"token_side: columns {s.start} to {s.start + s.size} of a table of {width}")
+        self.embedding = embedding
+
+    def weight_bytes(self):
+        return (self.gate.numel() + self.proj.numel()) * self.gate.element_size()
+
+    def reads_first(self):
+        return self.gate
+
+    def __call__(self, x, ctx):
+        s = self.spec
+        with section("side gate"):
+            z = ops.linear_act_rows(x, self.gate, "gelu_tanh", ctx.ids, self.embedding.side[:, s.start:s.start + s.size])
+        with section("side proj"):
+            return ops.linear(z, self.proj)
+
+
 @register_ffn("dense")
 class DenseFF(FeedForward):
     """down(act(up x)), no biases; the activation ("relu2": the square of relu, or "gelu_tanh") is a record field."""

@@ -4,7 +4,8 @@
     w_j = s[choice_j] / (sum_j s[choice_j] + 1e-20)
 Options of the record: s = sigmoid(z) element by element; a choice only among the experts of the best groups of
 neighbouring experts (a group's score: the sum of its largest choice scores); weights that are not divided by their
-sum; a constant factor on the weights.
+sum; a constant factor on the weights; no router at all, but an integer table that names every token id's experts,
+each with weight 1 / top (``route`` "table").
     y = sum_j w_j expert_{choice_j}(h)  (+ shared(h))
 The router's last ``identity`` outputs stand for experts that return h itself and have no tensors.  The experts are
 gated feed-forwards of one record (``parts/mlp.py``'s "gated" kind gives the formula); their matrices are stacked
@@ -44,12 +45,20 @@ class MixtureOfExperts(FeedForward):
             raise ValueError(f"{outputs} router outputs in {groups} groups of which {keep} are kept")
         if groups > 1 and spec.top > keep * (outputs // groups):
             raise ValueError(f"top {spec.top} of the {keep * (outputs // groups)} outputs of the kept groups")
+        self.by_table = getattr(spec, "route", "scores") == "table"
+        if getattr(spec, "route", "scores") not in ("scores", "table"):
+            raise ValueError(f"route {spec.route!r} is not built (known: scores, table)")
+        if self.by_table and spec.identity:
+            raise ValueError("experts by a table of token ids have no identity experts")
         self.shared = build_part("ffn", spec.shared, env) if spec.shared is not None else None
 
     @classmethod
     def param_infos(cls, spec):
         D, I, N = spec.hidden_size, spec.expert.intermediate_size, spec.experts + spec.identity
-        infos = {"router": ParamInfo((N, D), "vector"), "correction": ParamInfo((N,), "vector")}
+        if getattr(spec, "route", "scores") == "table":
+            infos = {spec.table_name: ParamInfo((spec.table_rows, spec.top), "table", below=spec.experts)}
+        else:
+            infos = {"router": ParamInfo((N, D), "vector"), "correction": ParamInfo((N,), "vector")}
         for e in range(spec.experts):
             infos[f"e{e}.gate"], infos[f"e{e}.up"] = ParamInfo((I, D)), ParamInfo((I, D))
             infos[f"e{e}.down"] = ParamInfo((D, I))
@@ -60,7 +69,10 @@ class MixtureOfExperts(FeedForward):
 
     def load(self, tensors):
         E = self.spec.experts
-        self.router, self.correction = tensors["router"], tensors["correction"]
+        if self.by_table:
+            self.table = tensors[self.spec.table_name].contiguous()
+        else:
+            self.router, self.correction = tensors["router"], tensors["correction"]
         # per expert [gate rows; up rows], all experts stacked
         self.gate_up = torch.stack([torch.cat([tensors[f"e{e}.gate"], tensors[f"e{e}.up"]], dim=0) for e in range(E)]).contiguous()
         self.down = torch.stack([tensors[f"e{e}.down"] for e in range(E)]).contiguous()
@@ -68,23 +80,31 @@ class MixtureOfExperts(FeedForward):
             self.shared.load({k[len("shared."):]: v for k, v in tensors.items() if k.startswith("shared.")})
 
     def weight_bytes(self):
-        n = (self.gate_up.numel() + self.down.numel()) * self.gate_up.element_size() + self.router.numel() * 4
+        n = (self.gate_up.numel() + self.down.numel()) * self.gate_up.element_size()
+        n += 0 if self.by_table else self.router.numel() * 4
         return n + (self.shared.weight_bytes() if self.shared is not None else 0)
 
     def __call__(self, x, ctx):
         s, ex = self.spec, self.spec.expert
         T = x.shape[0]
         with section("moe router"):
-            idx, weight = ops.moe_route(x, self.router, self.correction, s.top, getattr(s, "score", "softmax"),
-                                        getattr(s, "groups", 1), getattr(s, "group_keep", 1), getattr(s, "group_top", 2),
-                                        getattr(s, "route_scale", 1.0), getattr(s, "renormalize", True))
             # many pairs per expert (a prompt): tiles of 64 rows, where the bfloat16 kernel for them takes the sizes
             wide = (x.dtype == torch.bfloat16 and T * s.top >= 48 * s.experts and s.hidden_size % 8 == 0
                     and ex.intermediate_size % 8 == 0)
-            plan = ops.moe_plan(idx, s.experts, wide)
+            if self.by_table:
+                weight = None                              # every choice weighs 1 / top
+                idx, plan = ops.moe_plan_table(ctx.ids, self.table, s.experts, wide)
+            else:
+                idx, weight = ops.moe_route(x, self.router, self.correction, s.top, getattr(s, "score", "softmax"),
+                                            getattr(s, "groups", 1), getattr(s, "group_keep", 1), getattr(s, "group_top", 2),
+                                            getattr(s, "route_scale", 1.0), getattr(s, "renormalize", True))
+                plan = ops.moe_plan(idx, s.experts, wide)
         with section("moe experts"):
             gu = ops.moe_grouped_linear(x, self.gate_up, plan, T * s.top, gather_div=s.top)
             act = ops.gated_act(gu, ex.gate, None, ex.limit, ex.alpha)
+            if weight is None and s.top == 1 and self.shared is None:
+                # one expert of weight 1: its output is the token's
+                return ops.moe_grouped_linear(act, self.down, plan, T, scatter=True)
             pair_out = ops.moe_grouped_linear(act, self.down, plan, T * s.top, scatter=True, out_dtype=torch.float32)
         extra = self.shared(x, ctx) if self.shared is not None else None
         with section("moe combine"):

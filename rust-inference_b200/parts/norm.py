@@ -10,6 +10,8 @@ the mean squared deviation, float32.  It reads a residual of one or several stre
 absent: their plain sum), all in the same kernel."""
 from __future__ import annotations
 
+import torch
+
 from .. import ops
 from ..profiler import section
 from .base import Norm, Pending
@@ -68,13 +70,33 @@ class LayerNorm(Norm):
                                    out_w=out, read=read, rows=rows, bias=self.bias, more=more)
 
 
+def _single_stream(resid, delta):
+    """(the residual [tokens, width], what is pending as ``ops.rms_gains`` takes it: terms, entry, norm behind)."""
+    terms, entry, post = [], None, None
+    if isinstance(delta, Pending):
+        post = delta.post
+        if delta.mix is not None:
+            raise ValueError("rms_gains reads a residual of one stream without mixing weights")
+        if delta.y is not None:
+            terms = [(delta.y, delta.out)] + list(delta.more)
+        entry = delta.entry
+    elif delta is not None:
+        terms = [(delta, None)]
+    if resid.dim() == 3:
+        if resid.shape[1] != 1:
+            raise ValueError("rms_gains reads a residual of one stream")
+        resid = resid.view(resid.shape[0], resid.shape[2])
+    return resid, terms, entry, post
+
+
 @register_norm("rms_gains")
 class RMSGains(Norm):
     """RMS norm of the (single-stream) residual with one gain per name of the record: one pass computes
     1 / sqrt(mean(x^2) + eps) once and writes x times it times every gain.  The pending outputs (up to two, the sum of
     the two taken first: x + (a + b)) and the terms of a pass's entry (:class:`~.base.Injection`) join in the same
     pass, in float32; outputs that come with a norm behind their sublayer (``Pending.post``) are normed on the way.
-    ``one_plus``: the tensors hold the gains minus one, the gains are 1 + tensor.  Returns one tensor for one name, a tuple
+    ``one_plus``: the tensors hold the gains minus one, the gains are 1 + tensor; ``scalar``: they hold one number each,
+    spread over the row at load.  Returns one tensor for one name, a tuple
     for several."""
     graph_safe = True
     takes_hint = True
@@ -83,12 +105,14 @@ class RMSGains(Norm):
     def param_infos(cls, spec):
         # tensors that hold a gain minus one (``one_plus``) are drawn near 0 in the random-weights mode as well
         role = "vector" if getattr(spec, "one_plus", False) else "gain"
-        return {name: ParamInfo((spec.size,), role) for name in spec.names}
+        return {name: ParamInfo(() if getattr(spec, "scalar", False) else (spec.size,), role) for name in spec.names}
 
     def load(self, tensors):
         self.gains = tuple(tensors[name] for name in self.spec.names)
         if getattr(self.spec, "one_plus", False):
             self.gains = tuple((g + 1.0).contiguous() for g in self.gains)
+        if getattr(self.spec, "scalar", False):
+            self.gains = tuple(g.reshape(1).expand(self.spec.size).contiguous() for g in self.gains)
         if not 1 <= len(self.gains) <= 2:
             raise ValueError(f"rms_gains: {len(self.gains)} gains (one or two are built)")
 
@@ -96,21 +120,25 @@ class RMSGains(Norm):
         return sum(g.numel() * 4 for g in self.gains)
 
     def __call__(self, resid, delta=None, rows=None, then=None):
-        terms, entry, post = [], None, None
-        if isinstance(delta, Pending):
-            post = delta.post
-            if delta.mix is not None:
-                raise ValueError("rms_gains reads a residual of one stream without mixing weights")
-            if delta.y is not None:
-                terms = [(delta.y, delta.out)] + list(delta.more)
-            entry = delta.entry
-        elif delta is not None:
-            terms = [(delta, None)]
-        if resid.dim() == 3:
-            if resid.shape[1] != 1:
-                raise ValueError("rms_gains reads a residual of one stream")
-            resid = resid.view(resid.shape[0], resid.shape[2])
+        resid, terms, entry, post = _single_stream(resid, delta)
         with section("rmsnorm"):
             outs = ops.rms_gains(resid, self.gains, self.spec.eps, self.env.dtype, terms=terms, entry=entry, rows=rows,
                                  then=then, post=post)
         return outs[0] if len(outs) == 1 else outs
+
+
+@register_norm("no_norm")
+class NoNorm(Norm):
+    """No norm in front: whatever is pending joins the residual (as for ``rms_gains``, and in the same kernel), and the
+    sublayer gets the new residual's rows in the compute dtype."""
+    graph_safe = True
+    takes_hint = True
+
+    def __call__(self, resid, delta=None, rows=None, then=None):
+        if rows is not None:
+            raise ValueError("no_norm hands over whole steps, not selected rows")
+        resid, terms, entry, post = _single_stream(resid, delta)
+        out = torch.empty(resid.shape, dtype=self.env.dtype, device=resid.device)
+        with section("residual"):
+            ops.rms_gains(resid, (), 0.0, self.env.dtype, terms=terms, entry=entry, post=post, out=out, then=then)
+        return out

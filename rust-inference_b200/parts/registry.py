@@ -26,10 +26,12 @@ class ParamInfo:
     role "matrix": kept in the compute dtype, random init N(0, 0.02);
     role "gain":   kept in float32, random init 1 + U(-0.1, 0.1);
     role "vector": kept in float32, random init N(0, 0.02) (biases, rates, small weights that enter float32 arithmetic);
-    role "table":  integer table, kept as int32, random init zeros.
+    role "table":  integer table, kept as int32, random init zeros, or with ``below`` > 0 numbers under it, the entries
+                   of a row all different (a row's length must not exceed it).
     """
     shape: Tuple[int, ...]
     role: str = "matrix"
+    below: int = 0
 
 
 def _register(family: str, kind: str):

@@ -2,7 +2,7 @@
 configuration and a seed, or the same tensors made on the device without a file.
 
 Matrices and the embedding are N(0, 0.02), norm gains (the per-head q/k norms
-included) 1 + U(-0.1, 0.1), integer tables zero.  A value is a function of
+included) 1 + U(-0.1, 0.1), integer tables zero (or numbers under a bound).  A value is a function of
 (seed, tensor name, element index) and of nothing else (``csrc/random_fill.cuh``):
 the host code and the device kernel give the same bits, a tensor's values do not
 depend on which other tensors exist, and any part of a tensor (a few rows of an
@@ -63,12 +63,27 @@ def _fill(out: torch.Tensor, key: int, first: int, kind: int, a: float, b: float
         raise RuntimeError(f"random fill: {lib.ri_last_error().decode(errors='replace')}")
 
 
+def _random_table(key: int, shape, below: int, first_row: int) -> torch.Tensor:
+    """Integers under ``below``: row r is a run of neighbours (modulo ``below``) that starts at a place drawn for r."""
+    rows, cols = shape[0], 1
+    for d in shape[1:]:
+        cols *= d
+    if cols > below:
+        raise ValueError(f"{cols} different numbers under {below} in a row of a table")
+    starts = [_mix64(key + first_row + r) % below for r in range(rows)]
+    table = (torch.tensor(starts, dtype=torch.int64)[:, None] + torch.arange(cols)) % below
+    return table.view(shape).to(torch.int32)
+
+
 def random_tensor(seed: int, name: str, shape, role: str, dtype: torch.dtype, device="cpu",
-                  first_row: int = 0) -> torch.Tensor:
+                  first_row: int = 0, below: int = 0) -> torch.Tensor:
     """The tensor ``name`` of the random model with this seed, made where ``device`` says.
-    ``shape`` with ``first_row`` > 0 gives rows first_row .. first_row + shape[0] - 1 of it."""
+    ``shape`` with ``first_row`` > 0 gives rows first_row .. first_row + shape[0] - 1 of it; ``below``: an integer table's
+    bound (:class:`~..parts.registry.ParamInfo`)."""
     shape = tuple(int(d) for d in shape)
     if role == "table":
+        if below > 0:
+            return _random_table(tensor_key(seed, name), shape, below, first_row).to(device)
         return torch.zeros(shape, dtype=torch.int32, device=device)
     if role not in ("matrix", "gain", "vector"):
         raise ValueError(f"unknown parameter role {role!r}")
@@ -87,7 +102,8 @@ def random_tensor(seed: int, name: str, shape, role: str, dtype: torch.dtype, de
 
 def random_tensors(expected: Dict[str, object], seed: int, dtype: torch.dtype, device="cpu") -> Dict[str, torch.Tensor]:
     """``expected``: name -> ParamInfo."""
-    return {n: random_tensor(seed, n, info.shape, info.role, dtype, device) for n, info in sorted(expected.items())}
+    return {n: random_tensor(seed, n, info.shape, info.role, dtype, device, below=info.below)
+            for n, info in sorted(expected.items())}
 
 
 def write_random_model(config: dict, seed: int, out_dir: str, dtype: str = "bfloat16") -> str:

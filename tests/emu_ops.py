@@ -16,7 +16,7 @@ __all__ = ["embed", "rmsnorm", "add_rows", "silu_mul", "linear_swiglu", "linear"
            "sample", "mark_seen", "stream_norm", "activation", "gate_heads", "linear_heads", "latent_prep", "gla_recurrent",
            "head_norm_gate", "linear_act", "scale_", "embed_pair_hash", "short_conv", "delta_rule_recurrent", "gated_act",
            "linear_gated", "moe_route", "moe_plan", "moe_grouped_linear", "moe_combine", "rms_gains", "qkv_prep", "softcap_",
-           "embed_same", "mlstm_gates", "scalar_decay_recurrent", "mlstm_head_norm_gate"]
+           "embed_same", "mlstm_gates", "scalar_decay_recurrent", "mlstm_head_norm_gate", "moe_plan_table", "linear_act_rows"]
 
 
 def embed(ids, table, scale=1.0, copies=1):
@@ -58,6 +58,10 @@ def activation(x, kind):
 
 def linear_act(x, w, act):
     return activation(linear(x, w), act)
+
+
+def linear_act_rows(x, w, act, ids, rows):
+    return (activation(linear(x, w), act).float() * rows[ids.long()].float()).to(x.dtype)
 
 
 def _gate(z, fn):
@@ -200,7 +204,7 @@ def qk_norm_rope_append(qkv, num_heads, num_kv_heads, head_dim, q_gain, k_gain, 
 
 
 def attention(q, k_pool, v_pool, page_table, seq_slot, seq_start, seq_len, max_new, scale, window=0, sink=None, chunk=0,
-              softcap=0.0):
+              softcap=0.0, dist_bias=None):
     T, H, Dh = q.shape
     KV, P = k_pool.shape[1], k_pool.shape[2]
     G = H // KV
@@ -220,6 +224,8 @@ def attention(q, k_pool, v_pool, page_table, seq_slot, seq_start, seq_len, max_n
                 s = (kk[:, h // G, :] @ q[t, h].float()) * scale
                 if softcap:
                     s = softcap * torch.tanh(s / softcap)
+                if dist_bias is not None:
+                    s = s + dist_bias[h, torch.clamp(pos - idx, max=dist_bias.shape[1] - 1)]
                 if sink is None:
                     p = torch.softmax(s, dim=0)
                 else:
@@ -307,7 +313,7 @@ def delta_rule_recurrent(qkv, q_col, k_col, v_col, proj, beta_col, z, dt_bias, a
     k = (k / torch.sqrt((k * k).sum(-1, keepdim=True) + 1e-6)).repeat_interleave(rep, dim=1)
     v = qkv[:, v_col:v_col + heads * vdim].view(T, heads, vdim)
     beta = torch.sigmoid(proj[:, beta_col:beta_col + heads].float())
-    g = torch.exp(-torch.exp(a_log)[None, :, None] * torch.nn.functional.softplus((z.float() + dt_bias).view(T, heads, dim)))
+    g = torch.exp(-torch.exp(a_log)[None, :, None] * torch.nn.functional.softplus((z.float() + dt_bias).view(T, heads, -1)))
     o = torch.zeros(T, heads, vdim)
     for b in range(seq_slot.numel()):
         S = state[int(seq_slot[b])]
@@ -376,6 +382,11 @@ def moe_plan(idx, experts, wide=False):
     return perm, tiles, torch.tensor([experts, off], dtype=torch.int32), 0
 
 
+def moe_plan_table(ids, table, experts, wide=False):
+    idx = table[ids.long()].contiguous()
+    return idx, moe_plan(idx, experts, wide)
+
+
 def moe_grouped_linear(a, w, plan, rows_out, gather_div=0, scatter=False, out_dtype=None):
     perm, tiles, meta, _ = plan
     y = torch.zeros(rows_out, w.shape[1], dtype=out_dtype or a.dtype)
@@ -394,7 +405,7 @@ def moe_combine(pair_out, idx, weight, x, experts, extra=None):
     for j in range(top):
         ident = (idx[:, j] >= experts)[:, None]
         v = torch.where(ident, x.float(), pair_out.view(T, top, D)[:, j])
-        y += weight[:, j:j + 1] * v
+        y += (1.0 / top if weight is None else weight[:, j:j + 1]) * v
     if extra is not None:
         y += extra.float()
     return y.to(x.dtype)
@@ -472,7 +483,8 @@ def mlstm_head_norm_gate(o, gates, gain, eps, g, out_dtype):
 
 
 def qkv_prep(proj, q_col, k_col, v_col, heads, kv_heads, Dp, Dk, bias, rope_table, rot, pairs, unit, eps, k_pool, v_pool,
-             page_table, tok_seq, tok_pos, seq_slot, write_kv=True, norm="", q_gain=None, k_gain=None, norm_eps=0.0):
+             page_table, tok_seq, tok_pos, seq_slot, write_kv=True, norm="", q_gain=None, k_gain=None, norm_eps=0.0,
+             q_factor=None, unit_v=False, Dv=0):
     T = proj.shape[0]
     x = proj.float()
     if bias is not None:
@@ -505,6 +517,10 @@ def qkv_prep(proj, q_col, k_col, v_col, heads, kv_heads, Dp, Dk, bias, rope_tabl
         return t
 
     q, k = unit_rms(turn(normed(q, q_gain))), unit_rms(turn(normed(k, k_gain)))
+    if q_factor is not None:
+        q = q * q_factor[tok_pos.long()][:, None, None]
+    if unit_v and v is not None:
+        v = v / torch.sqrt((v * v).sum(-1, keepdim=True) / (Dv or Dk) + eps)
     if write_kv:
         P = k_pool.shape[2]
         for t in range(T):
