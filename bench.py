@@ -18,14 +18,16 @@ steps end at exactly 4,096 tokens.  One JSON line is printed:
   points     decode tokens a second at batch 1 and 64 (device-timed), and the same through
              the Python entry point (e2e_b1, e2e_b64)
 
-    python bench.py --design ranudra|pitenex|kagatar|puratar [--size small|large]
+    python bench.py --design ranudra|pitenex|kagatar|puratar|zavevik [--size small|large]
 
 measures another design (Ranudra: latent attention, gated linear attention, hyper-connections; Pitenex: chunked attention
 with a sink beside the gated delta rule, dense and routed feed-forwards; Kagatar: three kinds of attention with biases
 beside a clamped-swish feed-forward behind two gains over one RMS statistic; Puratar: norms in front of and behind every
-sublayer, attention with a gate per head or beside the matrix memory of xLSTM, dense and routed feed-forwards) at layer
-sizes that resemble a real model's, beside a Qwen3 model of the same width and depth (Puratar: beside the Pitenex model
-of the same width and depth, the closest design): decode at batch 8 and a
+sublayer, attention with a gate per head or beside the matrix memory of xLSTM, dense and routed feed-forwards; Zavevik:
+norms behind the sublayers only, attention with a distance bias, borrowed keys and values, the delta rule with one decay
+per head, experts by token id, a token-fed sublayer) at layer
+sizes that resemble a real model's, beside a Qwen3 model of the same width and depth (Puratar and Zavevik: beside the
+Pitenex model of the same width and depth, the closest design): decode at batch 8 and a
 prompt step of 2,048 tokens, device-timed, and the device time of every section of both steps from eager runs with
 the section timers on, with the bytes or flops of the sections that have a roofline.  One JSON line.
 
@@ -349,9 +351,32 @@ def puratar_config(z) -> dict:
             "loop": {"start": 0, "stop": 2, "times": 1}, "layers": [both, routed] * (z["layers"] // 2)}
 
 
-DESIGNS = {"ranudra": ranudra_config, "pitenex": pitenex_config, "kagatar": kagatar_config, "puratar": puratar_config}
+def zavevik_config(z) -> dict:
+    """Layers that read the residual itself, in turns of three: attention with a distance bias (32 buckets up to 1,024
+    positions) and capped scores, the same with its own queries over the keys and values of the layer before, and the
+    gated delta rule with one decay per head (heads of 128 x 128, half as many as the attention has, a convolution of 4
+    taps); heads of 128, four query heads per key/value head.  Every layer has a routed feed-forward (16 experts of an
+    eighth of the dense width, 4 per token by a table of token ids) and takes in 256 elements of the token."""
+    D, H = z["width"], z["heads"]
+    G = max(1, H // 4)
+    inter = -(-(2 * z["ff"] // 3) // 256) * 256          # three matrices of a gated feed-forward against two
+    mlp = {"kind": "moe", "router": {"experts": 16, "top": 4}, "expert": {"ff": inter // 8}}
+    attn = {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0,
+            "q_temp": {"coef": 0.1, "every": 4096}, "bias_max": 1024, "bias_rows": 32}
+    delta = {"type": "delta", "mlp": mlp,
+             "mixer": {"heads": max(1, H // 2), "kv_heads": max(1, H // 4), "dim": 128, "vdim": 128, "conv": 4}}
+    layers = []
+    for i in range(0, z["layers"] // 3 * 3, 3):
+        layers += [{"type": "attention", "mixer": attn, "mlp": mlp},
+                   {"type": "attention", "mixer": dict(attn, kv_from=i), "mlp": mlp}, delta]
+    return {"architecture": "Zavevik", "vocab": z["vocab"], "width": D, "norm": {"eps": 1e-6}, "token_side": {"dim": 256},
+            "layers": layers}
+
+
+DESIGNS = {"ranudra": ranudra_config, "pitenex": pitenex_config, "kagatar": kagatar_config, "puratar": puratar_config,
+           "zavevik": zavevik_config}
 # the model that a design is measured beside, where it is not the Qwen3 model of equal size: the closest design
-BESIDE = {"puratar": "pitenex"}
+BESIDE = {"puratar": "pitenex", "zavevik": "pitenex"}
 
 
 def qwen3_like(z) -> dict:

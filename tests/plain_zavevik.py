@@ -51,7 +51,7 @@ def over_rms(x, eps):
 
 
 def distance_bucket(n, rows, far):
-    half = rows / 2
+    half = rows // 2
     if n < half:
         return n
     # (a hair is added so that a distance exactly on a border belongs to the row that starts there)
@@ -77,7 +77,9 @@ def attention(h, w, m, eps, k, v):
     temp = m.get("q_temp")
     if temp:
         q = q * np.asarray([query_factor(p, temp["coef"], temp["every"]) for p in range(n)])[:, None, None]
-    rows = np.asarray([distance_bucket(d, w["rel"].shape[0], m["bias_max"]) for d in range(n)])
+    bias = np.zeros((n, H))                                    # by distance; none without a largest distance
+    if m.get("bias_max"):
+        bias = w["rel"][[distance_bucket(d, w["rel"].shape[0], m["bias_max"]) for d in range(n)]]
     cap = m.get("softcap")
     out = np.zeros((n, H, v.shape[-1]), dtype=F64)
     for hd in range(H):
@@ -86,7 +88,7 @@ def attention(h, w, m, eps, k, v):
         if cap:
             s = cap * np.tanh(s / cap)
         for p in range(n):
-            z = s[p, :p + 1] + w["rel"][rows[p - np.arange(p + 1)], hd]
+            z = s[p, :p + 1] + bias[p - np.arange(p + 1), hd]
             e = np.exp(z - z.max())
             out[p, hd] = (e @ v[:p + 1, g]) / e.sum()
     return out.reshape(n, -1) @ w["o"].T
