@@ -752,7 +752,7 @@ attention_decode_stream_kernel(const bf16* __restrict__ q, const __grid_constant
                 for (int t = 0; t < 4; t++)
 #pragma unroll
                     for (int e = 0; e < 4; e++)
-                        s[t][e] = fmaf(ri_bias_at((e >> 1) ? b1 : b0, a.bias.len, d0 - (t * 8 + qc * 2 + (e & 1))), a.inv_scale, s[t][e]);
+                        s[t][e] = fmaf(__ldg(((e >> 1) ? b1 : b0) + (d0 - qc * 2) - (t * 8 + (e & 1))), a.inv_scale, s[t][e]);
             }
         }
         // ---- mask (only the pages at the ends of the visible range need it), maximum, weights ---------------
@@ -1115,7 +1115,7 @@ extern "C" int ri_attention_decode_parts(int max_chunks) {
 // parts = ri_attention_decode_parts(max_chunks).  max_chunks * 128 must cover the longest sequence of the step.
 // sink [H] float32 or null: a learned term per head that joins the softmax's denominator only (the merge adds it).
 // softcap > 0: score <- softcap * tanh(score / softcap) after the scale (0: none; the scale must then be positive).
-// dist_bias [H, bias_len] float32 or null: added to the score by the query's distance to the key (distance_bias.cuh).
+// dist_bias (float32, bias_len entries a head between their padding) or null: added to the score by the query's distance to the key (distance_bias.cuh).
 extern "C" int ri_attention_decode_cap(const void* q, const void* k_pool, const void* v_pool, void* out, float* o_part,
                                        float* ml_part, const int* page_table, const int* seq_slot, const int* seq_len,
                                        int seqs, int H, int KV, int Dh, int mpps, int page_size, int num_pages,

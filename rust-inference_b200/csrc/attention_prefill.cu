@@ -153,7 +153,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_
 #pragma unroll
             for (int e = 0; e < 4; e++) {
                 float val = (cap_raw > 0.0f ? ri_softcap(s[t][e], cap_raw, inv_cap) : s[t][e]) * scale_log2;
-                if (near) val = fmaf(ri_bias_at(bias_row, bias.len, my_pos[e >> 1] - (k0 + t * 8 + qc * 2 + (e & 1))), LOG2E, val);
+                if (near) val = fmaf(__ldg(bias_row + (my_pos[e >> 1] - k0 - qc * 2) - (t * 8 + (e & 1))), LOG2E, val);
                 else val += far_bias;
                 if (edge) {
                     int key = k0 + t * 8 + qc * 2 + (e & 1);
@@ -232,7 +232,7 @@ extern "C" int ri_attention_prefill_head_dim() { return PF_DH; }
 // q, out [tokens, H, Dh] bf16; max_new = the most tokens one sequence brings in this step;
 // sink [H] float32 or null: a learned term per head that joins the softmax's denominator only
 // softcap > 0: score <- softcap * tanh(score / softcap) after the scale (0: none; the scale must then be positive)
-// dist_bias [H, bias_len] float32 or null: added to the score by the query's distance to the key (distance_bias.cuh)
+// dist_bias (float32, bias_len entries a head between their padding) or null: added to the score by the query's distance to the key (distance_bias.cuh)
 extern "C" int ri_attention_prefill(const void* q, const void* k_pool, const void* v_pool, void* out,
                                     const int* page_table, const int* seq_slot, const int* seq_start,
                                     const int* seq_len, int seqs, int max_new, int H, int KV, int Dh, int mpps,

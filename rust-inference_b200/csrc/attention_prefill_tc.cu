@@ -197,6 +197,11 @@ __device__ __forceinline__ unsigned long long ffma2(unsigned long long a, unsign
     asm("fma.rn.f32x2 %0, %1, %2, %3;\n" : "=l"(d) : "l"(a), "l"(b), "l"(c));
     return d;
 }
+__device__ __forceinline__ unsigned long long fmul2(unsigned long long a, unsigned long long b) {
+    unsigned long long d;
+    asm("mul.rn.f32x2 %0, %1, %2;\n" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
 __device__ __forceinline__ unsigned long long fadd2(unsigned long long a, unsigned long long b) {
     unsigned long long d;
     asm("add.rn.f32x2 %0, %1, %2;\n" : "=l"(d) : "l"(a), "l"(b));
@@ -578,8 +583,29 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 if (lane == 0) asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(smem_u32(&tail.s_read[t][idx & 1])) : "memory");
                 if (work.cap_raw > 0.0f) {                            // a soft cap on the scores, before the mask
                     const float inv_cap = 1.0f / work.cap_raw;
+                    float far4[4];                                    // is every score of the warp far below the cap?
 #pragma unroll
-                    for (int i = 0; i < TC_BN; i++) s[i] = ri_softcap(s[i], work.cap_raw, inv_cap);
+                    for (int q4 = 0; q4 < 4; q4++) {
+                        far4[q4] = fabsf(s[q4 * 16 + 15]);
+#pragma unroll
+                        for (int i = 0; i < 15; i++) far4[q4] = fmaxf(far4[q4], fabsf(s[q4 * 16 + i]));
+                    }
+                    const bool far = fmaxf(fmaxf(far4[0], far4[1]), fmaxf(far4[2], far4[3])) > RI_SOFTCAP_SMALL * work.cap_raw;
+                    if (!__any_sync(0xffffffffu, far)) {
+                        const unsigned long long ic2 = pack2(inv_cap, inv_cap);
+#pragma unroll
+                        for (int i = 0; i < TC_BN; i += 2) {
+                            const unsigned long long x = pack2(s[i], s[i + 1]), y = fmul2(x, ic2), t2 = fmul2(y, y);
+                            unsigned long long p = ffma2(pack2(RI_TANH_A4, RI_TANH_A4), t2, pack2(RI_TANH_A3, RI_TANH_A3));
+                            p = ffma2(p, t2, pack2(RI_TANH_A2, RI_TANH_A2));
+                            p = ffma2(p, t2, pack2(RI_TANH_A1, RI_TANH_A1));
+                            p = fmul2(p, t2);
+                            unpack2(ffma2(p, x, x), s[i], s[i + 1]);
+                        }
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < TC_BN; i++) s[i] = ri_softcap(s[i], work.cap_raw, inv_cap);
+                    }
                 }
                 if (BIAS) {                                           // a distance bias, after the cap and before the mask
                     const float* brow = ri_bias_row(work.bias, it.h);
@@ -590,7 +616,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                         for (int i = 0; i < TC_BN; i++) s[i] += far_bias;
                     } else {
 #pragma unroll
-                        for (int i = 0; i < TC_BN; i++) s[i] = fmaf(ri_bias_at(brow, work.bias.len, d0 - i), work.inv_scale, s[i]);
+                        for (int i = 0; i < TC_BN; i++) s[i] = fmaf(__ldg(brow + d0 - i), work.inv_scale, s[i]);
                     }
                 }
                 // a block of keys needs the mask if some query of this tile does not see all of it
@@ -806,7 +832,7 @@ extern "C" int ri_attention_prefill_tc(const void* q, const void* k_pool, const 
                                        int page_size, int num_pages, float scale, int window, const float* sink,
                                        float softcap, const float* dist_bias, int bias_len, int* err_flag,
                                        cudaStream_t stream) {
-    // dist_bias [H, bias_len] float32 or null: added to the score by the query's distance to the key (distance_bias.cuh)
+    // dist_bias (float32, bias_len entries a head between their padding) or null: added to the score by the query's distance to the key (distance_bias.cuh)
     // softcap > 0: score <- softcap * tanh(score / softcap) after the scale (0: none)
     if (seqs == 0 || max_new == 0 || tokens == 0) return 0;
     RI_REQUIRE(softcap >= 0.0f, "attention_prefill_tc: a soft cap is positive (0: none), got %g", (double)softcap);

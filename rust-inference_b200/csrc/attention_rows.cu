@@ -100,7 +100,7 @@ __device__ __forceinline__ void ar_strip(const float* __restrict__ qs, float* __
         }
         if (bias_row) {
 #pragma unroll
-            for (int r = 0; r < R; r++) s[r] += ri_bias_at(bias_row + (size_t)r * bias_len, bias_len, distance);
+            for (int r = 0; r < R; r++) s[r] += ri_bias_at(bias_row + (size_t)r * ri_bias_pitch(bias_len), bias_len, distance);
         }
     }
     float corr[R], p[R];
@@ -300,7 +300,7 @@ static int ar_launch(const void* q, const void* k_pool, const void* v_pool, void
 // q, out [tokens, H, Dh]; max_new = the most tokens one sequence brings in this step
 // sink [H] float32 or null: a learned term per head that joins the softmax's denominator only
 // softcap > 0: score <- softcap * tanh(score / softcap) after the scale (0: none)
-// dist_bias [H, bias_len] float32 or null: added to the score by the query's distance to the key (distance_bias.cuh)
+// dist_bias (float32, bias_len entries a head between their padding) or null: added to the score by the query's distance to the key (distance_bias.cuh)
 extern "C" int ri_attention_rows(const void* q, const void* k_pool, const void* v_pool, void* out, const int* page_table,
                                  const int* seq_slot, const int* seq_start, const int* seq_len, int seqs, int max_new,
                                  int H, int KV, int Dh, int mpps, int page_size, int num_pages, float scale, int window,

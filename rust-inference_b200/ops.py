@@ -947,14 +947,23 @@ def _sink(sink: Optional[torch.Tensor], heads: int) -> Optional[int]:
     return sink.data_ptr()
 
 
+DIST_BIAS_PAD = 192          # entries on either side of a head's row (csrc/distance_bias.cuh)
+
+
+def pad_distance_bias(bias: torch.Tensor) -> torch.Tensor:
+    """A bias by distance [heads, n] as the attention kernels take it: every row between copies of its first and its
+    last entry."""
+    return torch.cat([bias[:, :1].expand(-1, DIST_BIAS_PAD), bias, bias[:, -1:].expand(-1, DIST_BIAS_PAD)], dim=1).contiguous()
+
+
 def _bias(dist_bias: Optional[torch.Tensor], heads: int):
-    """(pointer, entries per head) of a distance bias [heads, n], (None, 0) for none."""
+    """(pointer, entries per head) of a padded distance bias [heads, pad + n + pad], (None, 0) for none."""
     if dist_bias is None:
         return None, 0
     _need(dist_bias, "dist_bias", torch.float32)
-    if dist_bias.dim() != 2 or dist_bias.shape[0] != heads or dist_bias.shape[1] < 1:
+    if dist_bias.dim() != 2 or dist_bias.shape[0] != heads or dist_bias.shape[1] <= 2 * DIST_BIAS_PAD:
         raise KernelError(f"attention: distance bias {tuple(dist_bias.shape)} does not fit {heads} heads")
-    return dist_bias.data_ptr(), dist_bias.shape[1]
+    return dist_bias.data_ptr(), dist_bias.shape[1] - 2 * DIST_BIAS_PAD
 
 
 def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_table: torch.Tensor,
@@ -967,7 +976,8 @@ def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_
     order that depends on its own position only, so the result does not depend on the step's cutting.
     ``sink`` [H] (float32): exp(sink[h]) joins head h's softmax denominator, with no key and no value.
     ``softcap`` > 0: score <- softcap * tanh(score / softcap) after the scale.
-    ``dist_bias`` [H, n] (float32): added to the score after that, entry min(distance, n - 1) of the head's row.
+    ``dist_bias`` (float32, from ``pad_distance_bias``): added to the score after that, entry min(distance, n - 1) of the
+    head's row of n.
     ``v_pool`` may be ``k_pool`` itself (values that are the keys: latent attention)."""
     _need(q, "q")
     tokens, H, Dh = q.shape

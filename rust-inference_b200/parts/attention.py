@@ -186,7 +186,7 @@ class Attention(Mixer):
         if s.sink:
             self.sink = tensors[sink]
         if self.bias_rows:
-            self.dist_bias = spread_over_distances(tensors[s.bias_name], s.bias_far)
+            self.dist_bias = ops.pad_distance_bias(spread_over_distances(tensors[s.bias_name], s.bias_far))
 
     def weight_bytes(self):
         return (self.qkv.numel() + self.o.numel()) * self.qkv.element_size()

@@ -12,6 +12,8 @@ import math
 import numpy as np
 import torch
 
+from rust_inference_b200.ops import DIST_BIAS_PAD
+
 __all__ = ["embed", "rmsnorm", "add_rows", "silu_mul", "linear_swiglu", "linear", "qk_norm_rope_append", "attention", "argmax",
            "sample", "mark_seen", "stream_norm", "activation", "gate_heads", "linear_heads", "latent_prep", "gla_recurrent",
            "head_norm_gate", "linear_act", "scale_", "embed_pair_hash", "short_conv", "delta_rule_recurrent", "gated_act",
@@ -225,7 +227,7 @@ def attention(q, k_pool, v_pool, page_table, seq_slot, seq_start, seq_len, max_n
                 if softcap:
                     s = softcap * torch.tanh(s / softcap)
                 if dist_bias is not None:
-                    s = s + dist_bias[h, torch.clamp(pos - idx, max=dist_bias.shape[1] - 1)]
+                    s = s + dist_bias[h, DIST_BIAS_PAD + torch.clamp(pos - idx, max=dist_bias.shape[1] - 2 * DIST_BIAS_PAD - 1)]
                 if sink is None:
                     p = torch.softmax(s, dim=0)
                 else:

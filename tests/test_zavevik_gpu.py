@@ -145,7 +145,7 @@ def test_attention_with_a_distance_bias(D, Hq, KV, rows, far, cap, dtype):
     for h in range(Hq):
         rel[(rows // 2 + h) % rows, h] += 7.0                       # which row stands out differs from head to head
     starts = bucket_starts(rows, far)
-    wide = spread_over_distances(_t(rel), far)
+    wide = ops.pad_distance_bias(spread_over_distances(_t(rel), far))
     bias = np.stack([[rel[P.distance_bucket(d, rows, far) if rows > 1 else 0, h] for d in range(n)] for h in range(Hq)])
     kp, vp, table = _paged(rng, kt, vt)
     args = (_np(qt), _np(kt), _np(vt), scale, cap)
@@ -191,7 +191,7 @@ def test_decode_with_a_distance_bias_over_a_batch(D):
     rng = np.random.default_rng(D)
     lengths, Hq, KV, scale = [1, 33, 700, 32, 411], 4, 2, 0.3
     bias = rng.standard_normal((Hq, 130)) * 2.0
-    wide = _t(bias)
+    wide = ops.pad_distance_bias(_t(bias))
     pages = sum(-(-n // 32) for n in lengths)
     kp = torch.zeros((pages, KV, 32, D), dtype=torch.bfloat16, device=DEV)
     vp = torch.zeros_like(kp)
