@@ -29,11 +29,11 @@ _SIGNATURES = {
     "ri_slots_create": (_P, [_I]), "ri_slots_destroy": (None, [_P]), "ri_slots_alloc": (_I, [_P, _P]),
     "ri_slots_free": (_I, [_P, _I]), "ri_slots_is_live": (_I, [_P, _I]), "ri_slots_require_live": (_I, [_P, _I]),
     "ri_slots_live_count": (_I, [_P]), "ri_slots_check": (_I, [_P]),
-    "ri_pages_create": (_P, [_I] * 5), "ri_pages_destroy": (None, [_P]), "ri_pages_table": (_P, [_P]),
+    "ri_pages_create": (_P, [_I] * 6), "ri_pages_destroy": (None, [_P]), "ri_pages_table": (_P, [_P]),
     "ri_pages_free": (_I, [_P]), "ri_pages_len": (_I, [_P, _I]), "ri_pages_needed": (_I, [_P, _I, _I]),
     "ri_pages_extend": (_I, [_P, _I, _I, _P]), "ri_pages_release_behind_window": (_I, [_P, _I]),
     "ri_pages_release": (None, [_P, _I]), "ri_pages_check": (_I, [_P]), "ri_pages_take_dirty": (_I, [_P, _P, _I]),
-    "ri_cache_create": (_P, [_I, _I, _I, _I, _I, _P]), "ri_cache_destroy": (None, [_P]),
+    "ri_cache_create": (_P, [_I, _I, _I, _I, _I, _P, _P]), "ri_cache_destroy": (None, [_P]),
     "ri_cache_slots": (_P, [_P]), "ri_cache_group": (_P, [_P, _I]), "ri_cache_alloc_slot": (_I, [_P, _P]),
     "ri_cache_free_slot": (_I, [_P, _I]), "ri_cache_length": (_I, [_P, _I, _P]),
     "ri_cache_extend": (_I, [_P, _I, _P, _P, _P]), "ri_cache_after_step": (None, [_P, _I, _P]),
@@ -115,17 +115,18 @@ class PageTable:
     ``window`` > 0: only the last ``window`` keys are ever read again, so pages
     that lie wholly before them are released after every step.  ``window`` < 0: a
     mask of chunks of ``-window`` positions counted from the sequence's start; the
-    pages before the chunk of the next query are released.  ``handle``: a
+    pages before the chunk of the next query are released.  ``keep``: the pages of a
+    sequence's first ``keep`` tokens are never released while it lives.  ``handle``: a
     group of a whole cache, which that cache owns.
     """
 
     def __init__(self, num_slots: int, num_pages: int, max_pages_per_seq: int, page_size: int, window: int = 0,
-                 handle: Optional[int] = None):
+                 handle: Optional[int] = None, keep: int = 0):
         self.num_slots, self.num_pages = num_slots, num_pages
-        self.max_pages_per_seq, self.page_size, self.window = max_pages_per_seq, page_size, window
+        self.max_pages_per_seq, self.page_size, self.window, self.keep = max_pages_per_seq, page_size, window, keep
         self._owned = handle is None
         if handle is None:
-            handle = lib().ri_pages_create(num_slots, num_pages, max_pages_per_seq, page_size, window)
+            handle = lib().ri_pages_create(num_slots, num_pages, max_pages_per_seq, page_size, window, keep)
             if not handle:
                 _raise(1)
         self._h = handle
@@ -185,14 +186,16 @@ class HostCache:
     """Slots, one ``PageTable`` per group of layers and the sequences' lengths, as one
     C++ object: a step's growth is one call."""
 
-    def __init__(self, num_slots: int, num_pages: int, max_pages_per_seq: int, page_size: int, windows: Sequence[int]):
+    def __init__(self, num_slots: int, num_pages: int, max_pages_per_seq: int, page_size: int, windows: Sequence[int],
+                 keeps: Optional[Sequence[int]] = None):
         w = np.asarray(list(windows), dtype=np.int32)
-        self._h = lib().ri_cache_create(num_slots, num_pages, max_pages_per_seq, page_size, len(w), w.ctypes.data)
+        k = np.asarray([0] * len(w) if keeps is None else list(keeps), dtype=np.int32)
+        self._h = lib().ri_cache_create(num_slots, num_pages, max_pages_per_seq, page_size, len(w), w.ctypes.data, k.ctypes.data)
         if not self._h:
             _raise(1)
         self.slots = SlotAllocator(num_slots, handle=lib().ri_cache_slots(self._h))
         self.groups = [PageTable(num_slots, num_pages, max_pages_per_seq, page_size, int(win),
-                                 handle=lib().ri_cache_group(self._h, g)) for g, win in enumerate(w)]
+                                 handle=lib().ri_cache_group(self._h, g), keep=int(k[g])) for g, win in enumerate(w)]
         self.num_pages = num_pages
 
     def __del__(self):

@@ -1,7 +1,7 @@
 """The cache: a slot per sequence, keys and values per layer in pages, fixed-size
 state per sequence beside them.
 
-Layers with the same needs (kv heads, head size, window, values of their own or not) form a *group* with
+Layers with the same needs (kv heads, head size, window and kept first tokens, values of their own or not) form a *group* with
 pools and a page table of its own, so that, say, full-attention layers and
 sliding-window layers neither share pages nor waste them.  Pools are laid out
 [entries of the group, pages, kv_heads, page_size, head_dim] (one layer's slice
@@ -75,10 +75,10 @@ class Cache:
         by_need: Dict[tuple, List[int]] = {}
         for i, r in enumerate(self.requests):
             if r is not None and r.kv_heads > 0:
-                by_need.setdefault((r.kv_heads, r.head_dim, r.mask, r.shared_kv), []).append(i)
+                by_need.setdefault((r.kv_heads, r.head_dim, r.mask, r.shared_kv, r.kept), []).append(i)
         # the bookkeeping of slots, pages and lengths is one C++ object (csrc/host_cache.cpp)
         self.host = HostCache(num_slots, num_pages, self.max_pages_per_seq, page_size,
-                              [need[2] for need in by_need])
+                              [need[2] for need in by_need], [need[4] for need in by_need])
         self.slots = self.host.slots
         self._any_window = any(need[2] != 0 for need in by_need)
         for (need, entries), pages in zip(by_need.items(), self.host.groups):

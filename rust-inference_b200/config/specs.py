@@ -48,6 +48,18 @@ class NoNormSpec:
 
 
 @dataclass(frozen=True)
+class DynTanhSpec:
+    """y = tanh(alpha x) * gain + bias over ``size`` elements, element by element and without any statistic (Dynamic
+    Tanh): ``alpha`` one number, gain and bias vectors.  The three tensors' local names are ``weight_name``,
+    ``bias_name`` and ``alpha_name``."""
+    size: int
+    weight_name: str = ""
+    bias_name: str = ".b"
+    alpha_name: str = ".alpha"
+    kind: str = "dyn_tanh"
+
+
+@dataclass(frozen=True)
 class LayerNormSpec:
     """y = (x - mean) / sqrt(var + eps) * gain (+ bias) over ``size`` elements, var the mean squared deviation.
 
@@ -136,6 +148,12 @@ class AttentionSpec:
     serves distance n < h, and row h + floor(ln(n / h) / ln(bias_far / h) (bias_rows - h)), at most the last one, the
     distances from h on.  ``own_kv`` False: the layer has no projections of keys and values and reads the cache entry
     that another layer of the same head counts and sizes writes.
+
+    ``keep_first`` > 0 (beside a window): a query also sees the sequence's first ``keep_first`` tokens, however far behind.
+    ``maps`` 2: differential attention.  Every query head and every key head holds two vectors of ``head_dim`` side by side;
+    each pair is a softmax map of its own over the head's one value, and the two results a, b of a query head give
+    o = a - lam b, then o / sqrt(mean(o^2) + pair_eps) over the value's elements, times (1 - pair_diff), with one number
+    lam = exp(sum(lq1 lk1)) - exp(sum(lq2 lk2)) + pair_diff for the layer (``pair_names``: the four vectors of ``head_dim``).
     """
     hidden_size: int
     num_heads: int
@@ -166,6 +184,11 @@ class AttentionSpec:
     bias_far: float = 0.0
     bias_name: str = "rel"
     own_kv: bool = True
+    keep_first: int = 0
+    maps: int = 1
+    pair_diff: float = 0.0
+    pair_eps: float = 0.0
+    pair_names: Tuple[str, str, str, str] = ("lq1", "lk1", "lq2", "lk2")
 
 
 @dataclass(frozen=True)
@@ -286,6 +309,10 @@ class MoESpec:
     plus correction), and only experts of the ``group_keep`` best groups can be chosen.  ``renormalize`` False: the
     weights are the chosen scores as they are; ``route_scale`` multiplies them.
 
+    ``score`` "logits": the choice is among the router's outputs themselves, and the weights are the softmax over the
+    chosen outputs alone; there is no correction.  ``router_bias``: the tensor that is added to the router's outputs ("" for
+    none).
+
     ``route`` "table": no router; an integer table (tensor ``table_name`` [table_rows, top]) gives every token id its
     experts, each with weight 1 / top."""
     hidden_size: int
@@ -304,6 +331,7 @@ class MoESpec:
     route: str = "scores"
     table_rows: int = 0
     table_name: str = "table"
+    router_bias: str = ""
 
 
 @dataclass(frozen=True)
@@ -365,7 +393,9 @@ class SwiGLUSpec:
 class EmbeddingSpec:
     """h[t] = table[ids[t]] * scale; ``copies`` > 1: [tokens, copies, hidden] with every row that many times
     (a residual kept as several streams starts with all of them equal).  ``side_width`` > 0: a second table of token
-    rows of that width (tensor ``side_name``) from which the layers' ``token_side`` parts read their columns."""
+    rows of that width (tensor ``side_name``) from which the layers' ``token_side`` parts read their columns.
+    ``norm``: a norm's record; the scaled rows pass that norm before they become the residual (its tensors' local names
+    follow "norm")."""
     vocab_size: int
     hidden_size: int
     kind: str = "embedding"
@@ -373,6 +403,7 @@ class EmbeddingSpec:
     copies: int = 1
     side_width: int = 0
     side_name: str = "side"
+    norm: object = None
 
 
 @dataclass(frozen=True)
@@ -403,7 +434,7 @@ class HeadSpec:
 @dataclass(frozen=True)
 class LayerSpec:
     """One block: two sub-layers, each a norm followed by a part, each added to
-    the residual stream (``arrangement`` "prenorm").
+    the residual stream (``arrangement`` "prenorm"); ``ffn`` None (with ``ffn_norm`` None): the mixer alone.
 
     ``names`` maps the block's four parts to the prefixes their tensors carry in
     the checkpoint, e.g. {"mixer": "model.layers.0.self_attn."}.

@@ -37,6 +37,7 @@
 #include "mma_helpers.cuh"
 #include "softcap.cuh"
 #include "distance_bias.cuh"
+#include "pair_heads.cuh"
 #include <cuda.h>
 #include <float.h>
 
@@ -112,7 +113,7 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
                         float* __restrict__ o_part, float* __restrict__ ml_part, const int* __restrict__ page_table,
                         const int* __restrict__ seq_slot, const int* __restrict__ seq_len, int H, int KV, int mpps,
                         int num_pages, int max_chunks, float scale_log2, int window, int* __restrict__ err,
-                        float cap_raw, DistBias bias) {
+                        float cap_raw, DistBias bias, int keep) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     DecodeSmem& sm = *reinterpret_cast<DecodeSmem*>(smem_raw);
     float* comb = reinterpret_cast<float*>(smem_raw + sizeof(DecodeSmem));
@@ -120,7 +121,7 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
     const int len = seq_len[b];                      // keys 0 .. len-1; the query is at position len-1
     const int first_key = ri_first_visible(len - 1, window);
     const int c0 = chunk * AD_CHUNK;
-    if (c0 >= len || c0 + AD_CHUNK <= first_key) return;       // nothing of this chunk is visible
+    if (c0 >= len || (c0 + AD_CHUNK <= first_key && c0 >= keep)) return;       // nothing of this chunk is visible
     const int G = H / KV;
     const int rows_pass = G < AD_ROWS ? G : AD_ROWS;           // rows of the combine area
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -129,7 +130,7 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
     pdl_trigger_early();
 
     const int key0 = c0 + warp * AD_PAGE;
-    const bool page_live = key0 < len && key0 + AD_PAGE > first_key;
+    const bool page_live = key0 < len && (key0 + AD_PAGE > first_key || key0 < keep);
     int page = -1;
     if (page_live) {
         page = key0 / AD_PAGE < mpps ? page_table[(size_t)slot * mpps + key0 / AD_PAGE] : -1;    // past the row: as unmapped
@@ -218,7 +219,7 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
 #pragma unroll
             for (int e = 0; e < 4; e++) {
                 int key = key0 + t * 8 + qc * 2 + (e & 1);
-                bool vis = page >= 0 && key < len && key >= first_key;
+                bool vis = page >= 0 && ri_sees(key, len - 1, first_key, keep);
                 s[t][e] = vis ? s[t][e] * scale_log2 : -FLT_MAX;
                 if (bias.table && vis) {              // a distance bias, after the scale and the cap
                     const int row = g0 + quad + (e >> 1) * 8;
@@ -388,8 +389,9 @@ struct StreamCursor {
     int seg, at;       // where the list has this (sequence, kv head), and where this piece of it
     int part;          // which of the (sequence, kv head)'s pieces it is (the cursor that computes keeps this)
     int len, first_key;
-    int p, p_end;      // the page (index within the sequence) and the end of the piece
-    int ids_base;      // lane l holds the pool index of page ids_base + l of the sequence
+    RiRuns runs;       // which pages of the sequence the query sees
+    int p, p_end;      // the page (its place among those) and the end of the piece
+    int ids_base;      // lane l holds the pool index of the page at place ids_base + l
     int id_lane;
     int slot_row;      // the sequence's row of the page table
 };
@@ -398,7 +400,7 @@ struct StreamArgs {
     const int* page_table;
     const int* seq_slot;
     const int* seq_len;
-    int seqs, KV, mpps, num_pages, window, max_pages, parts;
+    int seqs, KV, mpps, num_pages, window, keep, max_pages, parts;
     int* err;
     float cap_raw;          // a soft cap on the scores in unscaled units (cap / scale), 0 for none
     DistBias bias;          // a distance bias per head on the scores (table null: none)
@@ -408,13 +410,20 @@ struct StreamArgs {
 
 __device__ __forceinline__ int warp_sum_int(int v) { return __reduce_add_sync(0xffffffffu, v); }
 
-// the pages that the query of a sequence of `len` keys sees: [p_first, p_first + n)
-__device__ __forceinline__ int stream_visible(int len, int window, int max_pages, int& first_key, int& p_first) {
+// how many pages the query of a sequence of `len` keys sees, and which (every one of them holds a key that it sees)
+__device__ __forceinline__ int stream_visible(int len, int window, int keep, int max_pages, int& first_key, RiRuns& runs) {
     first_key = ri_first_visible(len - 1, window);
-    p_first = first_key / AD_PAGE;
+    int p_first = first_key / AD_PAGE;
     int p_last = (len + AD_PAGE - 1) / AD_PAGE;
     p_last = p_last < max_pages ? p_last : max_pages;     // no partial result has a place beyond (the merge reports it)
-    return p_last > p_first ? p_last - p_first : 0;
+    p_first = p_first < p_last ? p_first : p_last;
+    runs = RiRuns::of(p_first, keep, AD_PAGE);
+    return p_last - runs.shift;
+}
+__device__ __forceinline__ int stream_visible(int len, int window, int keep, int max_pages) {
+    int first_key;
+    RiRuns runs;
+    return stream_visible(len, window, keep, max_pages, first_key, runs);
 }
 // How a list of `total` pages is cut into runs for `workers` warps: the first `more` runs have len + 1 pages, the
 // others len, which together is the whole list; a list too short for runs of ADS_MIN_PAGES pages everywhere
@@ -473,8 +482,8 @@ struct SeqTable {
 
 __device__ __forceinline__ void stream_load_ids(StreamCursor& c, const StreamArgs& a, int lane) {
     c.ids_base = c.p;
-    int pg = c.p + lane;
-    int id = (pg < c.p_end) ? (pg < a.mpps ? a.page_table[(size_t)c.slot_row * a.mpps + pg] : -1) : 0;
+    const int pg = c.runs.block(c.p + lane);
+    int id = (c.p + lane < c.p_end) ? (pg < a.mpps ? a.page_table[(size_t)c.slot_row * a.mpps + pg] : -1) : 0;
     if (id < 0 || id >= a.num_pages) {
         atomicExch(a.err, 4);
         id = 0;
@@ -486,11 +495,10 @@ __device__ __forceinline__ void stream_load_ids(StreamCursor& c, const StreamArg
 // IDS: the cursor is the one that copies, so it needs the pages' places in the pool.
 template <bool IDS, bool SMALL>
 __device__ __forceinline__ void stream_piece(StreamCursor& c, const StreamArgs& a, const SeqTable<SMALL>& t, int off, int rem, const StreamCut& cut, int lane) {
-    int p_first;
     c.len = t.len(c.b);
-    const int n = stream_visible(c.len, a.window, a.max_pages, c.first_key, p_first);
-    c.p = p_first + off;
-    c.p_end = min(p_first + n, c.p + rem);
+    const int n = stream_visible(c.len, a.window, a.keep, a.max_pages, c.first_key, c.runs);
+    c.p = off;
+    c.p_end = min(n, c.p + rem);
     c.rem = rem - (c.p_end - c.p);
     c.seg = a.KV * t.before(c.b) + c.kvh * n;
     c.at = c.seg + off;
@@ -577,8 +585,7 @@ attention_decode_stream_kernel(const bf16* __restrict__ q, const __grid_constant
     }
     __syncwarp();
     if (SMALL) {
-        int fk, pf;
-        int v = lane < a.seqs ? stream_visible(tab.lane_len, a.window, a.max_pages, fk, pf) : 0;
+        int v = lane < a.seqs ? stream_visible(tab.lane_len, a.window, a.keep, a.max_pages) : 0;
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
             const int up = __shfl_up_sync(0xffffffffu, v, o);
@@ -587,8 +594,7 @@ attention_decode_stream_kernel(const bf16* __restrict__ q, const __grid_constant
         tab.lane_through = v;
     } else {
         for (int b = threadIdx.x; b < a.seqs; b += 32 * WARPS) {
-            int fk, pf;
-            pre[b + 1] = stream_visible(a.seq_len[b], a.window, a.max_pages, fk, pf);
+            pre[b + 1] = stream_visible(a.seq_len[b], a.window, a.keep, a.max_pages);
         }
         __syncthreads();
         if (warp == 0) {
@@ -664,7 +670,7 @@ attention_decode_stream_kernel(const bf16* __restrict__ q, const __grid_constant
     // The kernel before this one wrote the queries and the newest key and value (the last page of each
     // sequence); the pages before that one were written by earlier steps and may be copied at once.
 #pragma unroll 1
-    while (more && in_flight < SLOTS && (ci.p + 1) * AD_PAGE < ci.len) issue();
+    while (more && in_flight < SLOTS && (ci.runs.block(ci.p) + 1) * AD_PAGE < ci.len) issue();
     // every block of this grid is on an SM from the start (one per SM), so the kernel after it (the merge: small
     // blocks that read the lengths and then wait) may come in at once
     if (live) cc.part = cut.owner(cc.at) - cut.owner(cc.seg);
@@ -705,7 +711,7 @@ attention_decode_stream_kernel(const bf16* __restrict__ q, const __grid_constant
             l_run[0] = l_run[1] = 0.0f;
             fresh = false;
         }
-        const int key0 = cc.p * AD_PAGE;
+        const int key0 = cc.runs.block(cc.p) * AD_PAGE;
         const int rows = min(AD_PAGE, cc.len - key0);
         // ---- S[16 rows, 32 keys] = Q K^T ----------------------------------------------------------------
         float s[4][4];
@@ -762,7 +768,7 @@ attention_decode_stream_kernel(const bf16* __restrict__ q, const __grid_constant
 #pragma unroll
                 for (int e = 0; e < 4; e++) {
                     int key = key0 + t * 8 + qc * 2 + (e & 1);
-                    if (key >= cc.len || key < cc.first_key) s[t][e] = -FLT_MAX;
+                    if (!ri_sees(key, cc.len - 1, cc.first_key, a.keep)) s[t][e] = -FLT_MAX;
                 }
         }
         float mx[2] = {-FLT_MAX, -FLT_MAX};
@@ -901,28 +907,39 @@ struct MergeCut {
 // out[b, h, :] = the partial results of the head's chunks (or pieces) added up.  The block's four warps each take
 // a quarter of them (in rising order, four head elements per lane), then the four sums are added in
 // warp order: the order of the additions depends on the partial results' number only.
-__global__ void __launch_bounds__(AD_MERGE_THREADS)
+// MAPS 2 (differential attention): a block of twice as many warps merges two neighbouring heads, the two maps of one head,
+// and puts them together (pair_heads.cuh) before anything is rounded: out [seqs, H / 2, pair.width].
+template <int MAPS>
+__global__ void __launch_bounds__(AD_MERGE_THREADS* MAPS)
 attention_decode_merge_kernel(const float* __restrict__ o_part, const float* __restrict__ ml_part,
                               bf16* __restrict__ out, const int* __restrict__ seq_len, int H, int max_chunks,
-                              int window, MergeCut cut, const float* __restrict__ sink, int* __restrict__ err) {
+                              int window, int keep, MergeCut cut, const float* __restrict__ sink, PairOut pair,
+                              int* __restrict__ err) {
     constexpr int MW = AD_MERGE_THREADS / 32;            // warps
     constexpr int PER = (AD_DH + 127) / 128;             // float4 per lane
-    const int h = blockIdx.x, b = blockIdx.y;
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    __shared__ float s_w[AD_MERGE_TILE], s_red[MW], s_l[MW];
-    __shared__ int s_cnt[2][MW];
+    const int map = MAPS == 1 ? 0 : (int)threadIdx.x / AD_MERGE_THREADS, tid = (int)threadIdx.x - map * AD_MERGE_THREADS;
+    const int h = blockIdx.x * MAPS + map, b = blockIdx.y;
+    const int lane = tid & 31, warp = tid >> 5;
+    __shared__ float s_ws[MAPS][AD_MERGE_TILE], s_reds[MAPS][MW], s_ls[MAPS][MW];
+    __shared__ int s_cnts[MAPS][2][MW];
+    float *s_w = s_ws[map], *s_red = s_reds[map], *s_l = s_ls[map];
+    int(*s_cnt)[MW] = s_cnts[map];
     pdl_trigger();
     const int len = seq_len[b];                          // a table of the step, not the work of the kernel before
     const int first_key = ri_first_visible(len - 1, window);
     int c_lo = first_key / AD_CHUNK, c_hi = (len + AD_CHUNK - 1) / AD_CHUNK;           // [c_lo, c_hi)
     const bool too_long = c_hi > max_chunks;
     int stride = max_chunks;                             // partial results a head has room for
+    RiRuns runs;                                         // which chunks have results: place c is chunk runs.block(c)
     if (too_long) {
         // the caller's scratch memory has no partial results for the keys past max_chunks * 128: they are left
         // out (nothing is read past the sequence's rows) and the mistake is reported
         c_hi = max_chunks;
         c_lo = c_lo < c_hi ? c_lo : c_hi;
     }
+    runs = RiRuns::of(c_lo, keep, AD_CHUNK);
+    c_hi -= runs.shift;
+    c_lo = 0;
 #if ADS_OK
     if (cut.workers > 0) {
         // the streaming kernel's cut, from the same lengths: the pages before this sequence's and all pages
@@ -930,14 +947,12 @@ attention_decode_merge_kernel(const float* __restrict__ o_part, const float* __r
         int below = 0, all = 0;
         if (cut.seqs <= 32) {
             // every warp for itself: a lane per sequence, two additions across the warp
-            int f2, p2;
-            const int n = lane < cut.seqs ? stream_visible(seq_len[lane], window, max_pages, f2, p2) : 0;
+            const int n = lane < cut.seqs ? stream_visible(seq_len[lane], window, keep, max_pages) : 0;
             all = warp_sum_int(n);
             below = warp_sum_int(lane < b ? n : 0);
         } else {
-            for (int s = threadIdx.x; s < cut.seqs; s += AD_MERGE_THREADS) {
-                int f2, p2;
-                const int n = stream_visible(seq_len[s], window, max_pages, f2, p2);
+            for (int s = tid; s < cut.seqs; s += AD_MERGE_THREADS) {
+                const int n = stream_visible(seq_len[s], window, keep, max_pages);
                 all += n;
                 below += s < b ? n : 0;
             }
@@ -955,12 +970,11 @@ attention_decode_merge_kernel(const float* __restrict__ o_part, const float* __r
                 all += s_cnt[1][w];
             }
         }
-        int f2, p2;
-        const int n = stream_visible(len, window, max_pages, f2, p2);
-        const StreamCut runs(cut.KV * all, cut.workers);
+        const int n = stream_visible(len, window, keep, max_pages);
+        const StreamCut pieces(cut.KV * all, cut.workers);
         const int seg = cut.KV * below + (h / (H / cut.KV)) * n;
-        c_lo = 0;
-        c_hi = n > 0 ? runs.owner(seg + n - 1) - runs.owner(seg) + 1 : 0;
+        runs.kept = runs.shift = 0;                      // piece i stands at place i
+        c_hi = n > 0 ? pieces.owner(seg + n - 1) - pieces.owner(seg) + 1 : 0;
         stride = cut.parts;
     }
 #endif
@@ -968,7 +982,8 @@ attention_decode_merge_kernel(const float* __restrict__ o_part, const float* __r
     if (too_long && threadIdx.x == 0) atomicExch(err, 7);
     const float* ml = ml_part + ((size_t)b * H + h) * stride * 2;
     const float* op = o_part + ((size_t)b * H + h) * stride * AD_DH;
-    __shared__ __align__(16) float s_acc[MW][AD_DH];
+    __shared__ __align__(16) float s_accs[MAPS][MW][AD_DH];
+    float(*s_acc)[AD_DH] = s_accs[map];
     // The partial outputs of this warp's first eight chunks are asked for at once, before the maxima (on which
     // their weights depend) are known: the kernel is a chain of trips to L2, and this takes one out of it.
     float4 first[8][PER];
@@ -979,11 +994,11 @@ attention_decode_merge_kernel(const float* __restrict__ o_part, const float* __r
 #pragma unroll
         for (int j = 0; j < PER; j++) {
             const int d = (j * 32 + lane) * 4;
-            if (lo0 + u < hi0 && d < AD_DH) first[u][j] = ld_cg_f32x4(op + (size_t)(c_lo + lo0 + u) * AD_DH + d);
+            if (lo0 + u < hi0 && d < AD_DH) first[u][j] = ld_cg_f32x4(op + (size_t)runs.block(c_lo + lo0 + u) * AD_DH + d);
         }
     // the maximum over the visible chunks
     float M = -FLT_MAX;
-    for (int c = c_lo + (int)threadIdx.x; c < c_hi; c += AD_MERGE_THREADS) M = fmaxf(M, ld_cg_f32(ml + c * 2));
+    for (int c = c_lo + tid; c < c_hi; c += AD_MERGE_THREADS) M = fmaxf(M, ld_cg_f32(ml + runs.block(c) * 2));
     M = warp_max(M);
     if (lane == 0) s_red[warp] = M;
     __syncthreads();
@@ -997,14 +1012,14 @@ attention_decode_merge_kernel(const float* __restrict__ o_part, const float* __r
     for (int t0 = c_lo; t0 < c_hi; t0 += AD_MERGE_TILE) {
         const int n = min(AD_MERGE_TILE, c_hi - t0);
         __syncthreads();
-        for (int i = threadIdx.x; i < n; i += AD_MERGE_THREADS) {
-            float m = ld_cg_f32(ml + (t0 + i) * 2);
+        for (int i = tid; i < n; i += AD_MERGE_THREADS) {
+            float m = ld_cg_f32(ml + runs.block(t0 + i) * 2);
             s_w[i] = m == -FLT_MAX ? 0.0f : exp2f(m - M);
         }
         __syncthreads();
         // this warp's quarter of the tile
         const int lo = n * warp / MW, hi = n * (warp + 1) / MW;
-        for (int i = lo + lane; i < hi; i += 32) L += ld_cg_f32(ml + (t0 + i) * 2 + 1) * s_w[i];
+        for (int i = lo + lane; i < hi; i += 32) L += ld_cg_f32(ml + runs.block(t0 + i) * 2 + 1) * s_w[i];
         // eight chunks' partial outputs are asked for before the first is added (the additions stay in rising order
         // of the chunks)
         for (int i0 = lo; i0 < hi; i0 += 8) {
@@ -1016,7 +1031,7 @@ attention_decode_merge_kernel(const float* __restrict__ o_part, const float* __r
                 for (int j = 0; j < PER; j++) {
                     const int d = (j * 32 + lane) * 4;
                     if (have) v[u][j] = first[u][j];
-                    else if (i0 + u < hi && d < AD_DH) v[u][j] = ld_cg_f32x4(op + (size_t)(t0 + i0 + u) * AD_DH + d);
+                    else if (i0 + u < hi && d < AD_DH) v[u][j] = ld_cg_f32x4(op + (size_t)runs.block(t0 + i0 + u) * AD_DH + d);
                 }
 #pragma unroll
             for (int u = 0; u < 8; u++) {
@@ -1048,11 +1063,22 @@ attention_decode_merge_kernel(const float* __restrict__ o_part, const float* __r
     for (int w = 1; w < MW; w++) L += s_l[w];
     // a sink: one more term exp(sink[head]) in the denominator, with no key and no value (not scaled)
     if (sink && L > 0.0f) L += exp2f(sink[h] * 1.4426950408889634f - M);
-    for (int d = threadIdx.x; d < AD_DH; d += AD_MERGE_THREADS) {
+    for (int d = tid; d < AD_DH; d += AD_MERGE_THREADS) {
         float a = s_acc[0][d];
 #pragma unroll
         for (int w = 1; w < MW; w++) a += s_acc[w][d];
-        out[((size_t)b * H + h) * AD_DH + d] = __float2bfloat16_rn(L > 0.0f ? a / L : 0.0f);
+        a = L > 0.0f ? a / L : 0.0f;
+        if (MAPS == 1) out[((size_t)b * H + h) * AD_DH + d] = __float2bfloat16_rn(a);
+        else s_acc[0][d] = a;                            // (no other thread reads this column of this map before the barrier)
+    }
+    if (MAPS == 2) {
+        __shared__ float red[33];
+        static_assert(AD_DH <= 2 * AD_MERGE_THREADS, "a thread per head element");
+        __syncthreads();
+        const int d = threadIdx.x;
+        const float o = d < pair.vdim ? s_accs[0][0][d] - pair.lam * s_accs[MAPS - 1][0][d] : 0.0f;
+        const float f = pair.gain / sqrtf(block_sum(o * o, red) / (float)pair.vdim + pair.eps);
+        if (d < pair.width) out[((size_t)b * gridDim.x + blockIdx.x) * pair.width + d] = __float2bfloat16_rn(o * f);
     }
 }
 
@@ -1102,6 +1128,16 @@ static int launch_stream(int blocks, cudaStream_t stream, const bf16* q, const C
 }
 #endif
 
+static void launch_merge(const float* o_part, const float* ml_part, bf16* out, const int* seq_len, int seqs, int H, int max_chunks,
+                         int window, int keep, MergeCut cut, const float* sink, PairOut pair, int* err_flag, cudaStream_t stream) {
+    if (pair.on)
+        ri_launch_pdl(attention_decode_merge_kernel<2>, dim3(H / 2, seqs), dim3(2 * AD_MERGE_THREADS), 0, stream, o_part, ml_part,
+                      out, seq_len, H, max_chunks, window, keep, cut, sink, pair, err_flag);
+    else
+        ri_launch_pdl(attention_decode_merge_kernel<1>, dim3(H, seqs), dim3(AD_MERGE_THREADS), 0, stream, o_part, ml_part, out,
+                      seq_len, H, max_chunks, window, keep, cut, sink, pair, err_flag);
+}
+
 // how many partial results per (sequence, head) the scratch memory of ri_attention_decode must have room for
 extern "C" int ri_attention_decode_parts(int max_chunks) {
 #if ADS_OK && !defined(AD_NO_STREAM)
@@ -1116,12 +1152,21 @@ extern "C" int ri_attention_decode_parts(int max_chunks) {
 // sink [H] float32 or null: a learned term per head that joins the softmax's denominator only (the merge adds it).
 // softcap > 0: score <- softcap * tanh(score / softcap) after the scale (0: none; the scale must then be positive).
 // dist_bias (float32, bias_len entries a head between their padding) or null: added to the score by the query's distance to the key (distance_bias.cuh).
+// keep: beside a window, the sequence's first keys that every query sees.  pair_width > 0: heads 2 h and 2 h + 1 are the two
+// maps of differential attention; out [seqs, H / 2, pair_width] is their difference, normed (pair_heads.cuh).
 extern "C" int ri_attention_decode_cap(const void* q, const void* k_pool, const void* v_pool, void* out, float* o_part,
                                        float* ml_part, const int* page_table, const int* seq_slot, const int* seq_len,
                                        int seqs, int H, int KV, int Dh, int mpps, int page_size, int num_pages,
                                        int max_chunks, float scale, int window, const float* sink, float softcap,
-                                       const float* dist_bias, int bias_len, int* err_flag, cudaStream_t stream) {
+                                       const float* dist_bias, int bias_len, int keep, int pair_width, int pair_vdim,
+                                       float pair_lam, float pair_eps, float pair_gain, int* err_flag, cudaStream_t stream) {
     if (seqs == 0) return 0;
+    RI_REQUIRE(keep >= 0, "attention_decode: %d kept keys", keep);
+    if (window <= 0) keep = 0;                 // nothing is out of sight, or the mask is one of chunks
+    RI_REQUIRE(!pair_width || (H % 2 == 0 && (H / KV) % 2 == 0 && pair_vdim > 0 && pair_vdim <= Dh && pair_vdim <= pair_width &&
+                               pair_width <= 2 * AD_MERGE_THREADS && !sink),
+               "attention_decode: pairs of %d heads over %d kv heads, %d of %d elements in rows of %d", H, KV, pair_vdim, Dh, pair_width);
+    const PairOut pair{pair_width > 0 ? 1 : 0, pair_lam, pair_eps, pair_gain, pair_vdim, pair_width};
     RI_REQUIRE(softcap >= 0.0f && (softcap == 0.0f || scale > 0.0f), "attention_decode: a soft cap %g with scale %g", (double)softcap, (double)scale);
     const float cap_raw = softcap > 0.0f ? softcap / scale : 0.0f;
     RI_REQUIRE(!dist_bias || bias_len > 0, "attention_decode: a distance bias needs its length");
@@ -1159,6 +1204,7 @@ extern "C" int ri_attention_decode_cap(const void* q, const void* k_pool, const 
         a.max_pages = max_pages;
         a.parts = ADS_PARTS(max_chunks);
         a.window = window;
+        a.keep = keep;
         a.err = err_flag;
         a.cap_raw = cap_raw;
         a.bias = bias;
@@ -1183,8 +1229,7 @@ extern "C" int ri_attention_decode_cap(const void* q, const void* k_pool, const 
         cut.seqs = seqs;
         cut.KV = KV;
         cut.parts = a.parts;
-        ri_launch_pdl(attention_decode_merge_kernel, dim3(H, seqs), dim3(AD_MERGE_THREADS), 0, stream,
-                      (const float*)o_part, (const float*)ml_part, (bf16*)out, seq_len, H, max_chunks, window, cut, sink, err_flag);
+        launch_merge(o_part, ml_part, (bf16*)out, seq_len, seqs, H, max_chunks, window, keep, cut, sink, pair, err_flag, stream);
         RI_CHECK_LAUNCH("attention_decode_merge");
         return 0;
     }
@@ -1195,15 +1240,14 @@ extern "C" int ri_attention_decode_cap(const void* q, const void* k_pool, const 
     dim3 grid(max_chunks, KV, seqs);
     ri_launch_pdl(attention_decode_kernel, grid, dim3(32 * AD_WARPS), smem, stream,
                   (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, o_part, ml_part, page_table, seq_slot, seq_len,
-                  H, KV, mpps, num_pages, max_chunks, scale * 1.4426950408889634f, window, err_flag, cap_raw, bias);
+                  H, KV, mpps, num_pages, max_chunks, scale * 1.4426950408889634f, window, err_flag, cap_raw, bias, keep);
     RI_CHECK_LAUNCH("attention_decode");
     MergeCut chunks_of_128;
     chunks_of_128.workers = 0;
     chunks_of_128.seqs = seqs;
     chunks_of_128.KV = KV;
     chunks_of_128.parts = max_chunks;
-    ri_launch_pdl(attention_decode_merge_kernel, dim3(H, seqs), dim3(AD_MERGE_THREADS), 0, stream,
-                  (const float*)o_part, (const float*)ml_part, (bf16*)out, seq_len, H, max_chunks, window, chunks_of_128, sink, err_flag);
+    launch_merge(o_part, ml_part, (bf16*)out, seq_len, seqs, H, max_chunks, window, keep, chunks_of_128, sink, pair, err_flag, stream);
     RI_CHECK_LAUNCH("attention_decode_merge");
     return 0;
 }
@@ -1215,7 +1259,7 @@ extern "C" int ri_attention_decode_sink(const void* q, const void* k_pool, const
                                         cudaStream_t stream) {
     return ri_attention_decode_cap(q, k_pool, v_pool, out, o_part, ml_part, page_table, seq_slot, seq_len, seqs, H, KV, Dh,
                                    mpps, page_size, num_pages, max_chunks, scale, window, sink, 0.0f, nullptr, 0,
-                                   err_flag, stream);
+                                   0, 0, 0, 0.0f, 0.0f, 0.0f, err_flag, stream);
 }
 
 extern "C" int ri_attention_decode(const void* q, const void* k_pool, const void* v_pool, void* out, float* o_part,

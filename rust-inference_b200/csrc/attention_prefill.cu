@@ -10,7 +10,8 @@
 // on the tile it falls into (position within the step's tokens), not on the batch.
 //
 // Token t of sequence b: q row seq_start[b] + t, position seq_len[b] - n_b + t,
-// where n_b = seq_start[b+1] - seq_start[b].  It sees keys max(0, pos-window+1)..pos.
+// where n_b = seq_start[b+1] - seq_start[b].  It sees keys max(0, pos-window+1)..pos
+// (and the sequence's first `keep` keys).
 //
 // Compile with -DRI_HEAD_DIM=<multiple of 16, at most 256>.  Page size is 32.
 // Formula: thanhauco/rust-inference src/attention.rs:4-8, 111-150.
@@ -42,14 +43,14 @@ struct __align__(16) PrefillSmem {
 // keys [kb*64, kb*64+63] of one kv head into buffer `buf`: two pages, 16 bytes per copy
 __device__ __forceinline__ void load_kv_block(PrefillSmem& sm, int buf, int kb, const bf16* __restrict__ k_pool,
                                               const bf16* __restrict__ v_pool, const int* __restrict__ table, int kvh,
-                                              int KV, int num_pages, int len, int key_lo, int* err, bool with_v = true) {
+                                              int KV, int num_pages, int len, int key_lo, int keep, int* err, bool with_v = true) {
     constexpr int VEC = PF_DH / 8;
     for (int i = threadIdx.x; i < PF_BN * VEC; i += blockDim.x) {
         int r = i / VEC, c = (i % VEC) * 8;
         int key = kb * PF_BN + r;
         // a page that lies wholly before the first key any query of the tile sees may have been given back by a
         // window group already: it is not looked up, its rows are zeros (and masked)
-        bool ok = key < len && (key / PF_PAGE + 1) * PF_PAGE > key_lo;
+        bool ok = key < len && ((key / PF_PAGE + 1) * PF_PAGE > key_lo || key / PF_PAGE * PF_PAGE < keep);
         size_t off = 0;
         if (ok) {
             int page = table[key / PF_PAGE];
@@ -70,7 +71,8 @@ attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_
                          bf16* __restrict__ out, const int* __restrict__ page_table, const int* __restrict__ seq_slot,
                          const int* __restrict__ seq_start, const int* __restrict__ seq_len, int H, int KV, int mpps,
                          int num_pages, float scale_log2, int window, const float* __restrict__ sink, int shared_kv,
-                         int v_dims, int* __restrict__ err, float cap_raw, DistBias bias) {
+                         int v_dims, int* __restrict__ err, float cap_raw, DistBias bias, int keep) {
+    // keep: beside a window, the sequence's first keys that every query sees
     // bias: a distance bias per head, added after the cap (in units of log2 here, like the scaled scores)
     // cap_raw > 0: a soft cap on the scores in unscaled units (cap / scale), applied before the scale and the mask.
     // shared_kv: the values are the keys (one pool given as both): the key tiles serve as value tiles, nothing is
@@ -88,7 +90,8 @@ attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_
     const int rows = min(PF_BM, n_new - r_base);
     const int pos_first = len - n_new + r_base, pos_last = pos_first + rows - 1;
     const int key_lo = ri_first_visible(pos_first, window);
-    const int kb_lo = key_lo / PF_BN, kb_hi = pos_last / PF_BN;
+    const RiRuns runs = RiRuns::of(key_lo / PF_BN, keep, PF_BN);
+    const int n_blocks = pos_last / PF_BN + 1 - runs.shift;
     const int kvh = h / (H / KV);
     const int* table = page_table + (size_t)seq_slot[b] * mpps;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -101,7 +104,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_
         const bf16* src = q + ((size_t)(t_begin + r_base + (ok ? r : 0)) * H + h) * PF_DH + c;
         cp_async16(&sm.q[r][c], src, ok);
     }
-    load_kv_block(sm, 0, kb_lo, k_pool, v_pool, table, kvh, KV, num_pages, len, key_lo, err, !shared_kv);
+    load_kv_block(sm, 0, runs.block(0), k_pool, v_pool, table, kvh, KV, num_pages, len, key_lo, keep, err, !shared_kv);
     cp_async_commit();
 
     float o[PF_DH / 8][4];
@@ -116,9 +119,10 @@ attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_
     const float* bias_row = bias.table ? ri_bias_row(bias, h) : nullptr;
     const float far_bias = bias.table ? __ldg(bias_row + bias.len - 1) * LOG2E : 0.0f;
 
-    for (int kb = kb_lo; kb <= kb_hi; kb++) {
-        const int buf = (kb - kb_lo) & 1;
-        if (kb < kb_hi) load_kv_block(sm, buf ^ 1, kb + 1, k_pool, v_pool, table, kvh, KV, num_pages, len, key_lo, err, !shared_kv);
+    for (int j = 0; j < n_blocks; j++) {
+        const int kb = runs.block(j), buf = j & 1;
+        if (j + 1 < n_blocks)
+            load_kv_block(sm, buf ^ 1, runs.block(j + 1), k_pool, v_pool, table, kvh, KV, num_pages, len, key_lo, keep, err, !shared_kv);
         cp_async_commit();
         cp_async_wait<1>();              // everything but the block just asked for has arrived
         __syncthreads();
@@ -158,7 +162,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_
                 if (edge) {
                     int key = k0 + t * 8 + qc * 2 + (e & 1);
                     int p = my_pos[e >> 1];
-                    bool vis = key <= p && key >= ri_first_visible(p, window);
+                    bool vis = ri_sees(key, p, ri_first_visible(p, window), keep);
                     val = vis ? val : -FLT_MAX;
                 }
                 s[t][e] = val;
@@ -237,9 +241,11 @@ extern "C" int ri_attention_prefill(const void* q, const void* k_pool, const voi
                                     const int* page_table, const int* seq_slot, const int* seq_start,
                                     const int* seq_len, int seqs, int max_new, int H, int KV, int Dh, int mpps,
                                     int page_size, int num_pages, float scale, int window, const float* sink,
-                                    int v_dims, float softcap, const float* dist_bias, int bias_len, int* err_flag,
+                                    int v_dims, float softcap, const float* dist_bias, int bias_len, int keep, int* err_flag,
                                     cudaStream_t stream) {
     if (seqs == 0 || max_new == 0) return 0;
+    RI_REQUIRE(keep >= 0, "attention_prefill: %d kept keys", keep);
+    if (window <= 0) keep = 0;                 // nothing is out of sight, or the mask is one of chunks
     RI_REQUIRE(softcap >= 0.0f && (softcap == 0.0f || scale > 0.0f), "attention_prefill: a soft cap %g with scale %g", (double)softcap, (double)scale);
     RI_REQUIRE(!dist_bias || bias_len > 0, "attention_prefill: a distance bias needs its length");
     RI_REQUIRE(Dh == PF_DH, "attention_prefill: built for head_dim %d, called with %d", PF_DH, Dh);
@@ -263,7 +269,7 @@ extern "C" int ri_attention_prefill(const void* q, const void* k_pool, const voi
     attention_prefill_kernel<<<grid, 32 * PF_WARPS, smem, stream>>>(
         (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, (bf16*)out, page_table, seq_slot, seq_start, seq_len,
         H, KV, mpps, num_pages, scale * 1.4426950408889634f, window, sink, shared_kv, v_dims, err_flag,
-        softcap > 0.0f ? softcap / scale : 0.0f, DistBias{dist_bias, bias_len});
+        softcap > 0.0f ? softcap / scale : 0.0f, DistBias{dist_bias, bias_len}, keep);
     RI_CHECK_LAUNCH("attention_prefill");
     return 0;
 }

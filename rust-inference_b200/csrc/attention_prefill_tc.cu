@@ -50,7 +50,7 @@
 // start on a multiple of 1024 bytes (the swizzle's period), else the kernel reports error 6.
 //
 // Token t of sequence b: q row seq_start[b] + t, position seq_len[b] - n_b + t;
-// it sees keys max(0, pos-window+1)..pos.  A query's result depends on its position
+// it sees keys max(0, pos-window+1)..pos and, beside a window, the sequence's first `keep` keys.  A query's result depends on its position
 // and its place in the step, not on the batch.
 //
 // Compile with -DRI_HEAD_DIM=64 or 128.  Page size is 32.
@@ -219,13 +219,13 @@ __device__ __forceinline__ float ex2_approx(float x) {
 struct TcPages {
     int id[2];
 };
-__device__ __forceinline__ TcPages tc_pages(const int* __restrict__ table, int kb, int len, int key_lo, int num_pages, int* err) {
+__device__ __forceinline__ TcPages tc_pages(const int* __restrict__ table, int kb, int len, int key_lo, int keep, int num_pages, int* err) {
     TcPages r;
 #pragma unroll
     for (int j = 0; j < 2; j++) {
         const int pg = kb * (TC_BN / TC_PAGE) + j;
         int id = -1;
-        if (pg * TC_PAGE < len && (pg + 1) * TC_PAGE > key_lo) {
+        if (pg * TC_PAGE < len && ((pg + 1) * TC_PAGE > key_lo || pg * TC_PAGE < keep)) {
             id = table[pg];
             if (id < 0 || id >= num_pages) {
                 atomicExch(err, 4);
@@ -281,7 +281,8 @@ struct TcItem {
     int h, kvh;
     int t_first;                 // the item's first row in q and out
     int len, rows, n_tiles;
-    int pos_first, pos_last, key_lo, kb_lo;
+    int pos_first, pos_last, key_lo;
+    RiRuns runs;                 // place j of the item's blocks of keys is block runs.block(j)
     int n_blocks;                // blocks of 64 keys that the item's last row reaches
     int n_blocks_0;              // ... that the first tile's last row reaches (128 positions earlier)
     const int* table;
@@ -291,7 +292,7 @@ struct TcWork {
     const int* seq_slot;
     const int* seq_start;
     const int* seq_len;
-    int seqs, H, KV, mpps, groups_max, n_items, window;
+    int seqs, H, KV, mpps, groups_max, n_items, window, keep;
     const float* sink;          // [H] or null: exp(sink[h]) joins head h's softmax denominator, with no key and no value
     float cap_raw;              // a soft cap on the scores in unscaled units (cap / scale), 0 for none
     DistBias bias;              // a distance bias per head on the scores (table null: none)
@@ -320,9 +321,9 @@ __device__ __forceinline__ bool tc_item(const TcWork& w, int k, TcItem& it) {
     it.pos_first = it.len - n_new + r_base;
     it.pos_last = it.pos_first + it.rows - 1;
     it.key_lo = ri_first_visible(it.pos_first, w.window);
-    it.kb_lo = it.key_lo / TC_BN;
-    it.n_blocks = it.pos_last / TC_BN - it.kb_lo + 1;
-    it.n_blocks_0 = it.n_tiles > 1 ? min(it.n_blocks, (it.pos_first + TC_BM - 1) / TC_BN - it.kb_lo + 1) : it.n_blocks;
+    it.runs = RiRuns::of(it.key_lo / TC_BN, w.keep, TC_BN);
+    it.n_blocks = it.pos_last / TC_BN + 1 - it.runs.shift;
+    it.n_blocks_0 = it.n_tiles > 1 ? min(it.n_blocks, (it.pos_first + TC_BM - 1) / TC_BN + 1 - it.runs.shift) : it.n_blocks;
     it.kvh = it.h / (w.H / w.KV);
     it.table = w.page_table + (size_t)w.seq_slot[b] * w.mpps;
     return true;
@@ -431,7 +432,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 for (int j = 0; j < it.n_blocks && !dead; j++) {
                     const int gj = kv_base + j, buf = gj % TC_STAGES;
                     const unsigned parity = (unsigned)((gj / TC_STAGES - 1) & 1);
-                    const TcPages pg = tc_pages(it.table, it.kb_lo + j, it.len, it.key_lo, num_pages, err);   // under the wait below
+                    const TcPages pg = tc_pages(it.table, it.runs.block(j), it.len, it.key_lo, work.keep, num_pages, err);   // under the wait below
                     if (gj >= TC_STAGES) wait(&tail.k_empty[buf], parity);
                     if (dead) break;
 #ifdef TC_TEST_DROP_COPY_LEN
@@ -555,13 +556,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 kv_base += it.n_blocks;
                 continue;
             }
-            const int len = it.len, kb_lo = it.kb_lo, key_lo = it.key_lo, pos_first = it.pos_first, pos_last = it.pos_last;
+            const int len = it.len, key_lo = it.key_lo, pos_first = it.pos_first, pos_last = it.pos_last;
             const int my_pos = pos_first + t * TC_BM + row;
             const int tile_first = pos_first + t * TC_BM, tile_last = min(tile_first + TC_BM - 1, pos_last);
             const bool real_row = t * TC_BM + row < it.rows;
             float m = -FLT_MAX, l = 0.0f;
             for (int j = 0; j < my_blocks; j++) {
-                const int kb = kb_lo + j, idx = c + j, gj = kv_base + j;
+                const int kb = it.runs.block(j), idx = c + j, gj = kv_base + j;
                 if (!dead && !tc_mbar_wait(&tail.s_full[t][idx & 1], (unsigned)((idx >> 1) & 1))) { atomicExch(err, 5); tail.dead = 1; }
                 dead = dead || tail.dead != 0;
                 tc_fence_after();
@@ -626,7 +627,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
                     for (int i = 0; i < TC_BN; i++) {
                         int key = kb * TC_BN + i;
-                        bool vis = key <= my_pos && key >= first_vis;
+                        bool vis = ri_sees(key, my_pos, first_vis, work.keep);
                         s[i] = vis ? s[i] : -FLT_MAX;
                     }
                 }
@@ -711,11 +712,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 if (kb * TC_BN < key_lo) {
                     // value rows before the first key that any query of the item sees: their page may not have been
                     // copied at all (given back by a window group), so the stage may hold anything there, and P = 0
-                    // times a NaN is a NaN: zeroed as above
+                    // times a NaN is a NaN: zeroed as above (the kept rows in front of them are seen, and stay)
                     if (!dead && !tc_mbar_wait(&tail.v_full[st], st_parity)) { atomicExch(err, 5); tail.dead = 1; dead = true; }
                     unsigned char* v_tile = v_tiles + st * TC_KV_BYTES;
                     const int head_bad = min(TC_BN, key_lo - kb * TC_BN);
-                    for (int r = row >> 3; r < head_bad; r += TC_BM / 8)
+                    for (int r = max(0, work.keep - kb * TC_BN) + (row >> 3); r < head_bad; r += TC_BM / 8)
 #pragma unroll
                         for (int sl = 0; sl < TC_SLABS; sl++)
                             *(uint4*)(v_tile + sl * TC_KV_SLAB + r * 128 + ((row & 7) << 4)) = make_uint4(0, 0, 0, 0);
@@ -830,11 +831,14 @@ extern "C" int ri_attention_prefill_tc(const void* q, const void* k_pool, const 
                                        const int* page_table, const int* seq_slot, const int* seq_start,
                                        const int* seq_len, int tokens, int seqs, int max_new, int H, int KV, int Dh, int mpps,
                                        int page_size, int num_pages, float scale, int window, const float* sink,
-                                       float softcap, const float* dist_bias, int bias_len, int* err_flag,
+                                       float softcap, const float* dist_bias, int bias_len, int keep, int* err_flag,
                                        cudaStream_t stream) {
+    // keep: beside a window, the sequence's first keys that every query sees
     // dist_bias (float32, bias_len entries a head between their padding) or null: added to the score by the query's distance to the key (distance_bias.cuh)
     // softcap > 0: score <- softcap * tanh(score / softcap) after the scale (0: none)
     if (seqs == 0 || max_new == 0 || tokens == 0) return 0;
+    RI_REQUIRE(keep >= 0, "attention_prefill_tc: %d kept keys", keep);
+    if (window <= 0) keep = 0;                 // nothing is out of sight, or the mask is one of chunks
     RI_REQUIRE(softcap >= 0.0f, "attention_prefill_tc: a soft cap is positive (0: none), got %g", (double)softcap);
     RI_REQUIRE(!dist_bias || bias_len > 0, "attention_prefill_tc: a distance bias needs its length");
     RI_REQUIRE(Dh == TC_DH, "attention_prefill_tc: built for head_dim %d, called with %d", TC_DH, Dh);
@@ -879,6 +883,7 @@ extern "C" int ri_attention_prefill_tc(const void* q, const void* k_pool, const 
     work.groups_max = groups_max;
     work.n_items = (int)n_items;
     work.window = window;
+    work.keep = keep;
     work.sink = sink;
     work.cap_raw = softcap > 0.0f ? softcap / scale : 0.0f;
     work.bias = DistBias{dist_bias, bias_len};

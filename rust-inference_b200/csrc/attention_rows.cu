@@ -24,7 +24,8 @@
 //   q, out  [tokens, H, Dh];  k_pool, v_pool [pages, KV, page_size, Dh]
 //   sequence b: slot seq_slot[b], new tokens seq_start[b] .. seq_start[b+1]-1 of the packed arrays,
 //   length seq_len[b] after the step; new token i sits at position seq_len[b] - n_b + i and sees keys
-//   max(0, pos-window+1) .. pos  (window 0: all keys 0..pos).  kv head = h / (H / KV).
+//   max(0, pos-window+1) .. pos  (window 0: all keys 0..pos) and, beside a window, the sequence's first `keep` keys.
+//   kv head = h / (H / KV).
 // A page index outside the pool (or -1) among the pages a tile needs: error word 4, the strip is left
 // out.  Pages wholly before the first key that the tile sees are not looked up (a window group may have
 // given them back).
@@ -35,7 +36,7 @@
 
 #define AR_WARPS 8
 #define AR_STRIP 32
-#define AR_MAX_DH 512
+#define AR_MAX_DH 640
 #define AR_MAX_TILE 16
 #define AR_SMEM_BUDGET (200 * 1024)
 
@@ -55,15 +56,16 @@ template <> struct ArVec<__nv_bfloat16> {
 __host__ __device__ inline int ar_key_pitch(int Dh, bool vec4) { return vec4 ? Dh + 4 : Dh + 1; }    // floats per staged key
 
 // One strip of keys for R (1 or 2) rows that follow each other in shared memory and see the same keys j_lo .. j_hi of
-// the strip: scores (lane j = key j), the online-softmax update of each row's maximum and sum, and the rows' outputs
+// the strip, except hole_lo .. hole_hi - 1 (between the kept first keys and the window; a key in the hole has weight 0):
+// scores (lane j = key j), the online-softmax update of each row's maximum and sum, and the rows' outputs
 // (a lane owns head elements lane, lane + 32, ...; the keys are added in rising order).
 template <bool VEC4, int R>
 __device__ __forceinline__ void ar_strip(const float* __restrict__ qs, float* __restrict__ accs, float* __restrict__ ms,
                                          float* __restrict__ ls, const float* __restrict__ ks, const float* __restrict__ vs,
-                                         int row, int Dh, int kpitch, int j_lo, int j_hi, float scale, float softcap, int lane,
+                                         int row, int Dh, int kpitch, int j_lo, int j_hi, int hole_lo, int hole_hi, float scale, float softcap, int lane,
                                          const float* __restrict__ bias_row, int bias_len, int distance) {
     // bias_row: the distance bias of the first row's head (the next row's follows it), or null; distance: of key `lane`
-    const bool mine = lane >= j_lo && lane <= j_hi;
+    const bool mine = lane >= j_lo && lane <= j_hi && !(lane >= hole_lo && lane < hole_hi);
     float s[R];
 #pragma unroll
     for (int r = 0; r < R; r++) s[r] = -INFINITY;
@@ -158,7 +160,7 @@ attention_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, con
                       T* __restrict__ out, const int* __restrict__ page_table, const int* __restrict__ seq_slot,
                       const int* __restrict__ seq_start, const int* __restrict__ seq_len, int H, int KV, int Dh,
                       int mpps, int page_size, int num_pages, int tile_q, int group_chunk, float scale, int window,
-                      const float* __restrict__ sink, float softcap, DistBias bias, int* __restrict__ err) {
+                      int keep, const float* __restrict__ sink, float softcap, DistBias bias, int* __restrict__ err) {
     extern __shared__ __align__(16) float ar_smem[];
     const int b = blockIdx.z;
     const int t_begin = seq_start[b], n_new = seq_start[b + 1] - t_begin;
@@ -196,8 +198,13 @@ attention_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, con
 
     // strips: 32 consecutive keys of one page (the last strip of a page may be shorter), at places that
     // depend on the page size only
-    int key0 = key_lo - (key_lo % page_size) % AR_STRIP;              // start of the strip that holds key_lo
+    const int window_strip = key_lo - (key_lo % page_size) % AR_STRIP;      // start of the strip that holds key_lo
+    int key0 = keep > 0 ? 0 : window_strip;
     while (key0 <= pos_last) {
+        if (key0 >= keep && key0 < window_strip) {                    // past the strips of the kept keys
+            key0 = window_strip;
+            continue;
+        }
         const int page_idx = key0 / page_size, in_page = key0 - page_idx * page_size;
         const int width = min(AR_STRIP, page_size - in_page);
         const int page = page_idx < mpps ? table[page_idx] : -1;
@@ -230,16 +237,21 @@ attention_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, con
             const int i = unit / pairs, g_first = 2 * (unit - i * pairs);
             const int pos = pos0 + i;
             const int first = ri_first_visible(pos, window);
-            const int j_lo = max(first - key0, 0), j_hi = min(pos - key0, width - 1);       // the token's keys in this strip
+            // the token's keys in this strip: from the window's first one (or, where kept keys are, from the strip's start)
+            // to its own; between the kept ones and the window lies a hole
+            const int hole_lo = max(keep - key0, 0), hole_hi = first - key0;
+            const int j_lo = hole_lo > 0 ? 0 : max(hole_hi, 0);
+            int j_hi = min(pos - key0, width - 1);
+            if (hole_hi > j_hi) j_hi = min(j_hi, hole_lo - 1);
             if (j_lo > j_hi) continue;                                // none: the rows' state stays as it is
             const int row_a = i * ng + g_first;
             const float* bias_row = bias.table ? ri_bias_row(bias, kvh * G + g0 + g_first) : nullptr;
             const int distance = pos - key0 - lane;
             if (g_first + 1 < ng)
-                ar_strip<VEC4, 2>(qs, accs, ms, ls, ks, vs, row_a, Dh, kpitch, j_lo, j_hi, scale, softcap, lane, bias_row,
+                ar_strip<VEC4, 2>(qs, accs, ms, ls, ks, vs, row_a, Dh, kpitch, j_lo, j_hi, hole_lo, hole_hi, scale, softcap, lane, bias_row,
                                   bias.len, distance);
             else
-                ar_strip<VEC4, 1>(qs, accs, ms, ls, ks, vs, row_a, Dh, kpitch, j_lo, j_hi, scale, softcap, lane, bias_row,
+                ar_strip<VEC4, 1>(qs, accs, ms, ls, ks, vs, row_a, Dh, kpitch, j_lo, j_hi, hole_lo, hole_hi, scale, softcap, lane, bias_row,
                                   bias.len, distance);
         }
         key0 += width;
@@ -260,7 +272,7 @@ attention_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, con
 static void ar_geometry(int G, int Dh, int max_new, bool vec4, int* tile_q, int* group_chunk, size_t* smem) {
     const size_t strip = (size_t)AR_STRIP * (ar_key_pitch(Dh, vec4) + Dh) * sizeof(float);
     const size_t per_row = (size_t)(2 * Dh + 2) * sizeof(float);
-    int rows_max = (int)((AR_SMEM_BUDGET - strip) / per_row);          // at least 17 (head size 512)
+    int rows_max = (int)((AR_SMEM_BUDGET - strip) / per_row);          // at least 7 (head size 640)
     int gc = G < rows_max ? G : rows_max;
     int tq = rows_max / gc;
     tq = tq > AR_MAX_TILE ? AR_MAX_TILE : tq;
@@ -274,7 +286,7 @@ static void ar_geometry(int G, int Dh, int max_new, bool vec4, int* tile_q, int*
 template <typename T, bool VEC4>
 static int ar_launch(const void* q, const void* k_pool, const void* v_pool, void* out, const int* page_table,
                      const int* seq_slot, const int* seq_start, const int* seq_len, int seqs, int max_new, int H, int KV,
-                     int Dh, int mpps, int page_size, int num_pages, float scale, int window, const float* sink,
+                     int Dh, int mpps, int page_size, int num_pages, float scale, int window, int keep, const float* sink,
                      float softcap, DistBias bias, int* err_flag, cudaStream_t stream) {
     int tile_q, group_chunk;
     size_t smem;
@@ -292,7 +304,7 @@ static int ar_launch(const void* q, const void* k_pool, const void* v_pool, void
     dim3 grid((max_new + tile_q - 1) / tile_q, (unsigned)gy, seqs);
     attention_rows_kernel<T, VEC4><<<grid, 32 * AR_WARPS, smem, stream>>>(
         (const T*)q, (const T*)k_pool, (const T*)v_pool, (T*)out, page_table, seq_slot, seq_start, seq_len, H, KV, Dh, mpps,
-        page_size, num_pages, tile_q, group_chunk, scale, window, sink, softcap, bias, err_flag);
+        page_size, num_pages, tile_q, group_chunk, scale, window, keep, sink, softcap, bias, err_flag);
     RI_CHECK_LAUNCH("attention_rows");
     return 0;
 }
@@ -304,9 +316,11 @@ static int ar_launch(const void* q, const void* k_pool, const void* v_pool, void
 extern "C" int ri_attention_rows(const void* q, const void* k_pool, const void* v_pool, void* out, const int* page_table,
                                  const int* seq_slot, const int* seq_start, const int* seq_len, int seqs, int max_new,
                                  int H, int KV, int Dh, int mpps, int page_size, int num_pages, float scale, int window,
-                                 const float* sink, float softcap, const float* dist_bias, int bias_len, int dtype,
+                                 const float* sink, float softcap, const float* dist_bias, int bias_len, int keep, int dtype,
                                  int* err_flag, cudaStream_t stream) {
     if (seqs == 0 || max_new == 0) return 0;
+    RI_REQUIRE(keep >= 0, "attention_rows: %d kept keys", keep);
+    if (window <= 0) keep = 0;                 // nothing is out of sight, or the mask is one of chunks
     RI_REQUIRE(seqs > 0 && max_new > 0 && H > 0 && KV > 0 && Dh > 0 && page_size > 0 && mpps > 0, "attention_rows: bad sizes");
     RI_REQUIRE(H % KV == 0, "attention_rows: %d heads are not a multiple of %d kv heads", H, KV);
     RI_REQUIRE(Dh <= AR_MAX_DH, "attention_rows: head_dim %d exceeds the limit %d", Dh, AR_MAX_DH);
@@ -318,7 +332,7 @@ extern "C" int ri_attention_rows(const void* q, const void* k_pool, const void* 
     const uintptr_t align = f32 ? 15 : 7;
     const bool vec4 = Dh % 4 == 0 && (((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool) & align) == 0;
 #define AR_GO(T, V) ar_launch<T, V>(q, k_pool, v_pool, out, page_table, seq_slot, seq_start, seq_len, seqs, max_new, H, KV, \
-                                    Dh, mpps, page_size, num_pages, scale, window, sink, softcap, bias, err_flag, stream)
+                                    Dh, mpps, page_size, num_pages, scale, window, keep, sink, softcap, bias, err_flag, stream)
     if (f32) return vec4 ? AR_GO(float, true) : AR_GO(float, false);
     return vec4 ? AR_GO(__nv_bfloat16, true) : AR_GO(__nv_bfloat16, false);
 #undef AR_GO

@@ -35,7 +35,9 @@ SOURCES: Dict[str, Tuple[str, ...]] = {
     "linear_f32": ("linear_f32.cu", "common.cuh"),
     "streams": ("streams.cu", "common.cuh"),
     "norm_gains": ("norm_gains.cu", "common.cuh", "linear_skinny_geometry.cuh"),
+    "dyn_tanh": ("dyn_tanh.cu", "common.cuh", "linear_skinny_geometry.cuh"),
     "qkv_prep": ("qkv_prep.cu", "common.cuh"),
+    "pair_heads": ("pair_heads.cu", "common.cuh", "pair_heads.cuh"),
     "latent_attention": ("latent_attention.cu", "common.cuh"),
     "gla": ("gla.cu", "common.cuh"),
     "mlstm": ("mlstm.cu", "common.cuh"),
@@ -43,13 +45,13 @@ SOURCES: Dict[str, Tuple[str, ...]] = {
     "delta_rule": ("delta_rule.cu", "common.cuh"),
     "moe": ("moe.cu", "common.cuh", "mma_helpers.cuh"),
     "sampling": ("sampling.cu", "common.cuh"),
-    "attention_decode": ("attention_decode.cu", "common.cuh", "mma_helpers.cuh", "softcap.cuh", "distance_bias.cuh"),
+    "attention_decode": ("attention_decode.cu", "common.cuh", "mma_helpers.cuh", "softcap.cuh", "distance_bias.cuh", "pair_heads.cuh"),
     "attention_prefill": ("attention_prefill.cu", "common.cuh", "mma_helpers.cuh", "softcap.cuh", "distance_bias.cuh"),
     "linear_skinny": ("linear_skinny.cu", "common.cuh", "mma_helpers.cuh", "linear_skinny_geometry.cuh"),
     "linear_stream_tc": ("linear_stream_tc.cu", "common.cuh", "mma_helpers.cuh"),
     "attention_prefill_tc": ("attention_prefill_tc.cu", "common.cuh", "mma_helpers.cuh", "softcap.cuh", "distance_bias.cuh"),
     "attention_decode_noalloc": ("attention_decode_noalloc.cu", "attention_decode_noalloc.h", "attention_decode.cu",
-                                 "common.cuh", "mma_helpers.cuh", "softcap.cuh", "distance_bias.cuh"),
+                                 "common.cuh", "mma_helpers.cuh", "softcap.cuh", "distance_bias.cuh", "pair_heads.cuh"),
     "random_fill": ("random_fill.cu", "common.cuh", "random_fill.cuh"),
     # host code only: the same random values as random_fill.cu gives on the device
     "host_random": ("host_random.cpp", "random_fill.cuh"),

@@ -111,11 +111,31 @@ __device__ __forceinline__ bool ri_mbar_wait(unsigned long long* bar, unsigned p
 // `pos` sees the last `window` keys (pos - window + 1 .. pos).  `window` < 0: a mask of chunks of -window positions
 // counted from position 0 of the sequence: the query sees the keys of its own chunk up to itself
 // (pos - pos % size .. pos).  0: every key up to pos.  Both bounds never decrease with pos.
+// Beside a window a query may also see the sequence's first `keep` keys, however far behind they are.  What a query (or a
+// tile of queries) has to walk is then two runs of pages, or blocks of keys: the kept ones, and those from the first
+// visible key on.  RiRuns numbers them through: place j is block j for j < kept, block j + shift after that (where nothing is
+// kept: kept 0 and shift the first block; where the runs meet: shift 0).
 __host__ __device__ __forceinline__ int ri_first_visible(int pos, int window) {
     if (window > 0) return pos - window + 1 > 0 ? pos - window + 1 : 0;
     if (window < 0) return pos < 0 ? 0 : pos - pos % (-window);
     return 0;
 }
+
+__host__ __device__ __forceinline__ bool ri_sees(int key, int pos, int first_visible, int keep) {
+    return key <= pos && (key >= first_visible || key < keep);
+}
+struct RiRuns {
+    int kept, shift;
+    // first: the block that holds the first visible key; unit: keys per block
+    __host__ __device__ __forceinline__ static RiRuns of(int first, int keep, int unit) {
+        const int k = (keep + unit - 1) / unit;
+        RiRuns r;
+        r.kept = k < first ? k : first;
+        r.shift = first - r.kept;
+        return r;
+    }
+    __host__ __device__ __forceinline__ int block(int j) const { return j < kept ? j : j + shift; }
+};
 
 __device__ __forceinline__ float ld_f(const float* p) { return *p; }
 __device__ __forceinline__ float ld_f(const __nv_bfloat16* p) { return __bfloat162float(*p); }

@@ -72,15 +72,15 @@ struct Slots {
 
 // ---- the pages of one group of layers ------------------------------------------------------------
 struct Pages {
-    int slots, pages, mpps, page_size, window;
+    int slots, pages, mpps, page_size, window, keep;
     std::vector<int32_t> table;          // [slots, mpps], -1: unmapped
     std::vector<int> lens;               // tokens stored per slot
     std::vector<int> first_mapped;       // logical pages below it were released (window)
     std::vector<int> free_list;          // back() is given out next: page 0 first
     std::vector<uint8_t> dirty;          // slots whose row changed since the last clear
 
-    Pages(int slots_, int pages_, int mpps_, int page_size_, int window_)
-        : slots(slots_), pages(pages_), mpps(mpps_), page_size(page_size_), window(window_),
+    Pages(int slots_, int pages_, int mpps_, int page_size_, int window_, int keep_)
+        : slots(slots_), pages(pages_), mpps(mpps_), page_size(page_size_), window(window_), keep(keep_),
           table((size_t)slots_ * mpps_, -1), lens(slots_, 0), first_mapped(slots_, 0), dirty(slots_, 0) {
         for (int p = pages - 1; p >= 0; p--) free_list.push_back(p);
     }
@@ -118,7 +118,8 @@ struct Pages {
         if (before) *before = (int)start;
         return RI_OK;
     }
-    // gives back the pages that no later query of slot s can see (groups with a window)
+    // gives back the pages that no later query of slot s can see (groups with a window); the pages that hold the
+    // sequence's first `keep` tokens stay, since every later query sees those
     int release_behind_window(int s) {
         if (window == 0) return 0;
         // oldest key the next query (at position lens[s]) reads: the last `window` keys, or, with a negative value,
@@ -126,7 +127,7 @@ struct Pages {
         const long long first_needed = window > 0 ? (long long)lens[s] - window + 1
                                                   : (long long)lens[s] - (long long)lens[s] % (-window);
         int32_t* r = row(s);
-        int n = 0, p = first_mapped[s];
+        int n = 0, p = std::max(first_mapped[s], (keep + page_size - 1) / page_size);
         while ((long long)(p + 1) * page_size <= first_needed) {
             if (r[p] >= 0) {
                 free_list.push_back(r[p]);
@@ -135,7 +136,7 @@ struct Pages {
             }
             p++;
         }
-        first_mapped[s] = p;
+        first_mapped[s] = p;             // (behind the pages that are kept)
         if (n) dirty[s] = 1;
         return n;
     }
@@ -184,9 +185,9 @@ struct HostCache {
     std::vector<int> stamp;              // per slot: the step that named it last (a slot twice in one step)
     int step = 0;
 
-    HostCache(int num_slots, int num_pages, int mpps_, int page_size_, int n_groups, const int* windows)
+    HostCache(int num_slots, int num_pages, int mpps_, int page_size_, int n_groups, const int* windows, const int* keeps)
         : slots(num_slots), lens(num_slots, 0), mpps(mpps_), page_size(page_size_), stamp(num_slots, 0) {
-        for (int g = 0; g < n_groups; g++) groups.emplace_back(num_slots, num_pages, mpps_, page_size_, windows[g]);
+        for (int g = 0; g < n_groups; g++) groups.emplace_back(num_slots, num_pages, mpps_, page_size_, windows[g], keeps[g]);
     }
     long long max_seq_len() const { return (long long)mpps * page_size; }
 
@@ -242,12 +243,16 @@ int ri_slots_live_count(void* h) { return as<Slots>(h)->n - (int)as<Slots>(h)->f
 int ri_slots_check(void* h) { return as<Slots>(h)->check(); }
 
 // ---- one group's pages alone ----------------------------------------------------------------------
-void* ri_pages_create(int slots, int pages, int mpps, int page_size, int window) {
+void* ri_pages_create(int slots, int pages, int mpps, int page_size, int window, int keep) {
     if (slots <= 0 || pages <= 0 || mpps <= 0 || page_size <= 0) {
         fail(RI_CACHE_ERROR, "page counts and the page size must be positive");
         return nullptr;
     }
-    return new Pages(slots, pages, mpps, page_size, window);
+    if (keep < 0) {
+        fail(RI_CACHE_ERROR, "a sequence's kept first tokens cannot be negative");
+        return nullptr;
+    }
+    return new Pages(slots, pages, mpps, page_size, window, keep);
 }
 void ri_pages_destroy(void* h) { delete as<Pages>(h); }
 int32_t* ri_pages_table(void* h) { return as<Pages>(h)->table.data(); }
@@ -272,7 +277,7 @@ int ri_pages_take_dirty(void* h, int* out, int cap) {
 }
 
 // ---- the whole cache ------------------------------------------------------------------------------
-void* ri_cache_create(int num_slots, int num_pages, int mpps, int page_size, int n_groups, const int* windows) {
+void* ri_cache_create(int num_slots, int num_pages, int mpps, int page_size, int n_groups, const int* windows, const int* keeps) {
     if (num_slots <= 0) {
         fail(RI_CACHE_ERROR, "the cache needs at least one slot");
         return nullptr;
@@ -281,7 +286,12 @@ void* ri_cache_create(int num_slots, int num_pages, int mpps, int page_size, int
         fail(RI_CACHE_ERROR, "page counts and the page size must be positive");
         return nullptr;
     }
-    return new HostCache(num_slots, num_pages, mpps, page_size, n_groups, windows);
+    for (int g = 0; g < n_groups; g++)
+        if (keeps[g] < 0) {
+            fail(RI_CACHE_ERROR, "a sequence's kept first tokens cannot be negative");
+            return nullptr;
+        }
+    return new HostCache(num_slots, num_pages, mpps, page_size, n_groups, windows, keeps);
 }
 void ri_cache_destroy(void* h) { delete as<HostCache>(h); }
 void* ri_cache_slots(void* h) { return &as<HostCache>(h)->slots; }

@@ -3,8 +3,9 @@
 // `moe_route`   per token: logits z = R x (float32), scores s = softmax(z) over all N outputs of the router (or the
 //               sigmoid of each), choice scores s + correction, optionally only within the best groups of neighbouring
 //               outputs (`MoeRule`), the `top` largest of them (ties: the lower index), and as weights the chosen
-//               outputs' scores s divided by their sum (+ 1e-20) or as they are, times a constant.  Every sum has a
-//               fixed order.
+//               outputs' scores s divided by their sum (+ 1e-20) or as they are, times a constant.  Or the choice is by
+//               the logits themselves and the weights are the softmax over the chosen ones alone.  The logits may have a
+//               bias.  Every sum has a fixed order.
 // `moe_plan`    the step's (token, choice) pairs grouped by expert: `perm` lists the pairs of expert 0, then of expert
 //               1 and so on (pairs whose choice is not one of the first E outputs, identity experts, are left out), and
 //               `tiles` cuts every expert's run into tiles of MOE_BM rows: (expert, first row in perm, rows).  One
@@ -38,20 +39,28 @@ __device__ __forceinline__ float4 moe_ld4(const bf16* p) {
 }
 
 // How scores become a choice and weights.  mode 0: scores are the softmax over all outputs; mode 1: the sigmoid of every
-// output on its own.  Choice scores are the scores plus the correction.  groups > 1: the outputs form `groups` equal runs
+// output on its own; mode 2: the logits themselves, without a correction, and the weights are the softmax over the chosen
+// outputs alone (times `scale`).  `bias` [N] (or null) is added to the logits first.  Choice scores are the scores plus the correction.  groups > 1: the outputs form `groups` equal runs
 // of neighbours, a run's score is the sum of its `gtop` largest choice scores, and only the outputs of the `keep` best
 // runs can be chosen (ties: the lower index, for runs as for outputs).  The weights are the chosen outputs' scores
 // (without the correction) times `scale`, divided by their sum first when `renorm` is set.
 struct MoeRule {
     int mode, groups, keep, gtop, renorm;
     float scale;
+    const float* bias;
 };
 
 // One warp: s [N] holds the logits on entry, c [N] and gs [groups] are scratch.
 __device__ __forceinline__ void moe_choose(float* s, float* c, float* gs, const float* __restrict__ correction,
                                            int* __restrict__ idx, float* __restrict__ weight, int t, int N, int top, int lane,
                                            const MoeRule rule) {
-    if (rule.mode == 0) {
+    if (rule.bias) {
+        for (int n = lane; n < N; n += 32) s[n] += rule.bias[n];
+        __syncwarp();
+    }
+    if (rule.mode == 2) {
+        for (int n = lane; n < N; n += 32) c[n] = s[n];
+    } else if (rule.mode == 0) {
         float mx = -INFINITY;
         for (int n = lane; n < N; n += 32) mx = fmaxf(mx, s[n]);
         mx = warp_max(mx);
@@ -142,7 +151,17 @@ __device__ __forceinline__ void moe_choose(float* s, float* c, float* gs, const 
         picked_sum += s[at];
         __syncwarp();
     }
-    if (lane == 0) {
+    if (lane == 0 && rule.mode == 2) {
+        // the first choice has the largest logit
+        float* w = weight + (size_t)t * top;
+        const float mx = w[0];
+        float sum = 0.0f;
+        for (int j = 0; j < top; j++) {
+            w[j] = expf(w[j] - mx);
+            sum += w[j];
+        }
+        for (int j = 0; j < top; j++) w[j] = w[j] / sum * rule.scale;
+    } else if (lane == 0) {
         const float div = rule.renorm ? picked_sum + 1e-20f : 1.0f;
         for (int j = 0; j < top; j++) weight[(size_t)t * top + j] = weight[(size_t)t * top + j] / div * rule.scale;
     }
@@ -253,14 +272,16 @@ moe_route_wide_kernel(const T* __restrict__ x, const float* __restrict__ router,
 
 extern "C" int ri_moe_route_rule(const void* x, const float* router, const float* correction, int* idx, float* weight,
                                  int tokens, int D, int N, int top, int mode, int groups, int keep, int gtop, float scale,
-                                 int renorm, int dtype, cudaStream_t stream) {
+                                 int renorm, const float* bias, int dtype, cudaStream_t stream) {
     if (tokens == 0) return 0;
-    RI_REQUIRE(mode == 0 || mode == 1, "moe_route: score rule %d", mode);
+    RI_REQUIRE(mode >= 0 && mode <= 2, "moe_route: score rule %d", mode);
+    RI_REQUIRE(mode == 2 || correction, "moe_route: score rule %d needs its correction", mode);
     RI_REQUIRE(groups >= 1 && N % groups == 0 && keep >= 1 && keep <= groups && gtop >= 1,
                "moe_route: %d outputs in %d groups of which %d are kept", N, groups, keep);
     RI_REQUIRE(top <= keep * (N / groups), "moe_route: top %d of the %d outputs of the kept groups", top, keep * (N / groups));
     MoeRule rule;
     rule.mode = mode; rule.groups = groups; rule.keep = keep; rule.gtop = gtop; rule.renorm = renorm; rule.scale = scale;
+    rule.bias = bias;
     RI_REQUIRE(tokens > 0 && D > 0 && N > 0 && top > 0 && top <= N, "moe_route: bad sizes (top %d of %d)", top, N);
     RI_REQUIRE(N <= 4096, "moe_route: %d router outputs (up to 4096 are built)", N);
     const size_t smem = (size_t)MOE_ROUTE_WARPS * (2 * N + groups) * sizeof(float);
@@ -738,5 +759,5 @@ extern "C" int ri_moe_combine(const float* pair_out, const int* idx, const float
 
 extern "C" int ri_moe_route(const void* x, const float* router, const float* correction, int* idx, float* weight,
                             int tokens, int D, int N, int top, int dtype, cudaStream_t stream) {
-    return ri_moe_route_rule(x, router, correction, idx, weight, tokens, D, N, top, 0, 1, 1, 1, 1.0f, 1, dtype, stream);
+    return ri_moe_route_rule(x, router, correction, idx, weight, tokens, D, N, top, 0, 1, 1, 1, 1.0f, 1, nullptr, dtype, stream);
 }

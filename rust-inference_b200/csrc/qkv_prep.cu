@@ -16,7 +16,9 @@
 // then, with `unit`, the head is divided by its root mean square over its Dk true elements:
 //     x' / sqrt(sum(x'^2) / Dk + eps)                    (no gain);
 // and q heads are multiplied by the position's factor, q_factor[pos] (float32 [factor_rows], null: none);
-// q goes to q_out, k to the token's place in its page.  v heads get their bias, are divided by their root mean square
+// q goes to q_out (with `maps` > 1 a q head holds that many queries of Dk / maps elements side by side, as the key heads do:
+// it goes out as `maps` heads [tokens, H maps, Dp], each with its own query's elements and zeros elsewhere, so that its
+// product with a whole key is the product with its own part of the key), k to the token's place in its page.  v heads get their bias, are divided by their root mean square
 // over their Dv true elements with `unit_v` (eps as for `unit`, no gain), and are stored.  All of it float32.
 #include "common.cuh"
 
@@ -39,6 +41,7 @@ struct QpArgs {
     int norm;
     float norm_eps;
     int H, KV, Dp, Dk, mpps, page_size, num_pages, write_kv;
+    int maps;
     int* err;
 };
 
@@ -109,7 +112,7 @@ __global__ void qkv_prep_kernel(QpArgs a) {
         const int col = (which == 0 ? a.q_col : (which == 1 ? a.k_col : a.v_col)) + hh * Dp;
         T* dst;
         if (which == 0) {
-            dst = (T*)a.q_out + ((size_t)t * H + h) * Dp;
+            dst = (T*)a.q_out + ((size_t)t * H + h) * a.maps * Dp;
         } else {
             if (page < 0) continue;
             dst = (T*)(which == 1 ? a.k_pool : a.v_pool) + (((size_t)page * KV + hh) * a.page_size + pos % a.page_size) * Dp;
@@ -158,6 +161,13 @@ __global__ void qkv_prep_kernel(QpArgs a) {
             inv = 1.0f / sqrtf(warp_sum(ss) / (float)a.Dk + a.eps);
         }
         if (which == 0) inv *= qf;
+        if (which == 0 && a.maps > 1) {
+            const int per = a.Dk / a.maps;
+            for (int m = 0; m < a.maps; m++)
+                for (int d = lane; d < Dp; d += 32) st_f(dst + (size_t)m * Dp + d, d / per == m ? x[d] * inv : 0.0f);
+            __syncwarp();
+            continue;
+        }
         for (int d = lane; d < Dp; d += 32) st_f(dst + d, x[d] * inv);
         __syncwarp();
     }
@@ -308,7 +318,7 @@ __global__ void qkv_prep_vec_kernel(QpArgs a, int group) {
                 const float4 b0 = *reinterpret_cast<const float4*>(a.bias + col), b1 = *reinterpret_cast<const float4*>(a.bias + col + 4);
                 x[0] += b0.x; x[1] += b0.y; x[2] += b0.z; x[3] += b0.w; x[4] += b1.x; x[5] += b1.y; x[6] += b1.z; x[7] += b1.w;
             }
-            if (which == 0) dst = (T*)a.q_out + ((size_t)t * H + h) * Dp + d0;
+            if (which == 0) dst = (T*)a.q_out + ((size_t)t * H + h) * a.maps * Dp + d0;
             else if (page >= 0)
                 dst = (T*)(which == 1 ? a.k_pool : a.v_pool) + (((size_t)page * KV + hh) * a.page_size + pos % a.page_size) * Dp + d0;
         }
@@ -358,7 +368,15 @@ __global__ void qkv_prep_vec_kernel(QpArgs a, int group) {
         }
 #pragma unroll
         for (int j = 0; j < 8; j++) x[j] *= inv;
-        if (dst) Qp8<T>::store(dst, x);
+        if (dst && which == 0 && a.maps > 1) {
+            const int per = a.Dk / a.maps;
+            for (int m = 0; m < a.maps; m++) {
+                float y[8];
+#pragma unroll
+                for (int j = 0; j < 8; j++) y[j] = d0 + j >= m * per && d0 + j < (m + 1) * per ? x[j] : 0.0f;
+                Qp8<T>::store(dst + (size_t)m * Dp, y);
+            }
+        } else if (dst) Qp8<T>::store(dst, x);
     }
 }
 
@@ -370,7 +388,7 @@ extern "C" int ri_qkv_prep_norm(const void* proj, long long ld, int q_col, int k
                                 const int* seq_slot, const float* rope_table, int rope_rows, int rot, int pairs, int unit,
                                 float eps, const float* q_gain, const float* k_gain, int norm, float norm_eps,
                                 const float* q_factor, int factor_rows, int unit_v, int Dv, int tokens, int H, int KV, int Dp,
-                                int Dk, int mpps, int page_size, int num_pages, int write_kv,
+                                int Dk, int mpps, int page_size, int num_pages, int write_kv, int maps,
                                 int dtype, int* err_flag, cudaStream_t stream) {
     if (tokens == 0) return 0;
     RI_REQUIRE(norm >= 0 && norm <= 2, "qkv_prep: norm %d", norm);
@@ -382,6 +400,7 @@ extern "C" int ri_qkv_prep_norm(const void* proj, long long ld, int q_col, int k
     RI_REQUIRE(!rope_table || rot > 0, "qkv_prep: a rotation table needs rotated elements");
     RI_REQUIRE(page_size > 0 && mpps > 0, "qkv_prep: bad page sizes");
     RI_REQUIRE(dtype == RI_DTYPE_F32 || dtype == RI_DTYPE_BF16, "qkv_prep: unknown dtype %d", dtype);
+    RI_REQUIRE(maps >= 1 && Dk % maps == 0, "qkv_prep: %d queries in heads of %d elements", maps, Dk);
     if (KV == 0) write_kv = 0;
     QpArgs a;
     a.proj = proj; a.ld = ld; a.q_col = q_col; a.k_col = k_col; a.v_col = v_col; a.bias = bias; a.q_out = q_out;
@@ -390,7 +409,7 @@ extern "C" int ri_qkv_prep_norm(const void* proj, long long ld, int q_col, int k
     a.q_factor = q_factor; a.factor_rows = factor_rows; a.unit_v = unit_v; a.Dv = Dv;
     a.q_gain = q_gain; a.k_gain = k_gain; a.norm = norm; a.norm_eps = norm_eps;
     a.pairs = pairs; a.unit = unit; a.eps = eps; a.H = H; a.KV = KV; a.Dp = Dp; a.Dk = Dk; a.mpps = mpps;
-    a.page_size = page_size; a.num_pages = num_pages; a.write_kv = write_kv; a.err = err_flag;
+    a.page_size = page_size; a.num_pages = num_pages; a.write_kv = write_kv; a.maps = maps; a.err = err_flag;
     const int heads_total = H + KV + (v_col >= 0 ? KV : 0);
     const int es = dtype == RI_DTYPE_F32 ? 4 : 2;
     // every piece of eight elements must start on 16 bytes: the row pitch, the columns, the heads and the pointers

@@ -177,7 +177,13 @@ class Model:
         return ask() if ask is not None else None
 
     def cache_requests(self):
-        reqs = [self.blocks[layer].mixer.cache_request() for layer in self.cache_entry_layers]
+        reqs = []
+        for entry, layer in enumerate(self.cache_entry_layers):
+            req = self.blocks[layer].mixer.cache_request()
+            others = [self.blocks[e.layer].mixer.cache_request() for e in self.spec.schedule
+                      if e.cache == entry and e.layer != layer]
+            others = [r for r in others if r is not None]
+            reqs.append(req.for_readers(others) if req is not None and others else req)
         if self.embed_cache_entry is not None:
             reqs.append(self._embed_request())
         return reqs

@@ -30,8 +30,8 @@ _SIGNATURES = {
     ("moe", "ri_moe_plan_table"): [_P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _P, _P],
     ("elementwise", "ri_embed_rows_same"): [_P, _P, _P, _L, _I, _I, _I, _I, _P, _P],
     ("norm_gains", "ri_norm_gains_post"): [_P] * 6 + [_P, _I, _F] + [_P] * 6 + [_I, _I, _F, _P, _F, _L, _I, _P, _I, _I, _P, _P],
-    ("qkv_prep", "ri_qkv_prep_norm"): [_P, _L, _I, _I, _I] + [_P] * 9 + [_I, _I, _I, _I, _F, _P, _P, _I, _F, _P, _I, _I, _I] + [_I] * 10 + [_P, _P],
-    ("moe", "ri_moe_route_rule"): [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P],
+    ("qkv_prep", "ri_qkv_prep_norm"): [_P, _L, _I, _I, _I] + [_P] * 9 + [_I, _I, _I, _I, _F, _P, _P, _I, _F, _P, _I, _I, _I] + [_I] * 11 + [_P, _P],
+    ("moe", "ri_moe_route_rule"): [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P],
     ("gla", "ri_gla_recurrent_scalar"): [_P, _L, _I, _I, _I, _P, _I, _I, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     ("mlstm", "ri_mlstm_gates"): [_P, _L, _I, _I, _P, _P, _F, _P, _P, _P, _P, _I, _I, _I, _I, _P],
     ("mlstm", "ri_mlstm_head_norm_gate"): [_P, _P, _P, _F, _P, _L, _P, _I, _I, _I, _I, _I, _P],
@@ -48,7 +48,7 @@ _SIGNATURES = {
     ("moe", "ri_moe_grouped_linear"): [_P, _L, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     ("moe", "ri_moe_combine"): [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
     ("rope_kv", "ri_qk_norm_rope_append_pairs"): [_P] * 10 + [_F, _P, _I, _I] + [_I] * 10 + [_P, _P],
-    ("latent_attention", "ri_latent_prep"): [_P, _L, _I, _I] + [_P] * 8 + [_F, _P] + [_I] * 11 + [_P, _P],
+    ("latent_attention", "ri_latent_prep"): [_P, _L, _I, _I] + [_P] * 8 + [_F, _P] + [_I] * 12 + [_P, _P],
     ("gla", "ri_gla_recurrent"): [_P, _L, _I, _I, _I, _P, _P, _F, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     ("gla", "ri_gla_head_norm_gate"): [_P, _P, _F, _P, _L, _P, _I, _I, _I, _I, _I, _P],
     ("linear_f32", "ri_linear_heads_f32"): [_P, _P, _P, _I, _I, _I, _I, _L, _L, _L, _L, _P],
@@ -56,24 +56,27 @@ _SIGNATURES = {
     ("elementwise", "ri_add_rows"): [_P, _P, _L, _I, _P],
     ("elementwise", "ri_silu_mul"): [_P, _P, _I, _I, _I, _I, _P],
     ("rope_kv", "ri_qk_norm_rope_append"): [_P] * 10 + [_F, _P, _I, _I] + [_I] * 9 + [_P, _P],
-    ("attention_rows", "ri_attention_rows"): [_P] * 8 + [_I] * 8 + [_F, _I, _P, _F, _P, _I, _I, _P, _P],
+    ("attention_rows", "ri_attention_rows"): [_P] * 8 + [_I] * 8 + [_F, _I, _P, _F, _P, _I, _I, _I, _P, _P],
     ("elementwise", "ri_softcap_f32"): [_P, _L, _F, _P],
     ("norm_gains", "ri_norm_gains"): [_P] * 6 + [_P, _I, _F] + [_P] * 6 + [_I, _I, _F, _I, _P, _I, _I, _P, _P],
+    ("dyn_tanh", "ri_dyn_tanh"): [_P] * 7 + [_I, _I, _I, _P, _I, _I, _P],
+    ("dyn_tanh", "ri_embed_dyn_tanh"): [_P, _P, _F, _P, _P, _P, _P, _I, _I, _I, _I, _P, _P],
+    ("pair_heads", "ri_pair_heads"): [_P, _P, _F, _F, _F, _I, _I, _I, _I, _I, _I, _P],
     ("linear_f32", "ri_linear_f32"): [_P, _P, _P, _I, _I, _I, _P],
     ("sampling", "ri_sample"): [_P, _L, _I, _I, _P, _P, _L, _P, _P, _P, _P, _P, _P, _P, _L, _I, _I, _P, _I, _P],
     ("sampling", "ri_sample_work_bytes"): [_I, _I],
     ("sampling", "ri_argmax"): [_P, _L, _I, _I, _P, _P, _P, _P],
     ("sampling", "ri_mark_seen"): [_P, _L, _P, _P, _I, _I, _P],
     ("attention_decode", "ri_attention_decode_sink"): [_P] * 9 + [_I] * 8 + [_F, _I, _P, _P, _P],
-    ("attention_decode", "ri_attention_decode_cap"): [_P] * 9 + [_I] * 8 + [_F, _I, _P, _F, _P, _I, _P, _P],
+    ("attention_decode", "ri_attention_decode_cap"): [_P] * 9 + [_I] * 8 + [_F, _I, _P, _F, _P, _I] + [_I, _I, _I, _F, _F, _F] + [_P, _P],
     ("linear_skinny", "ri_linear_skinny"): [_P, _P, _P, _I, _I, _I, _I, _I, _P, _P],
     ("linear_skinny", "ri_linear_skinny_act"): [_P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P],
     ("linear_skinny", "ri_linear_skinny_gated"): [_P, _P, _P, _I, _I, _I, _I, _P, _P],
     ("linear_skinny", "ri_linear_skinny_gated_with"): [_P, _P, _P, _I, _I, _I, _I, _F, _F, _P, _P],
     ("linear_stream_tc", "ri_linear_stream_tc"): [_P, _P, _P, _I, _I, _I, _I, _I, _P, _P],
     ("linear_stream_tc", "ri_linear_stream_tc_gate"): [_P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P, _P],
-    ("attention_prefill_tc", "ri_attention_prefill_tc"): [_P] * 8 + [_I] * 9 + [_F, _I, _P, _F, _P, _I, _P, _P],
-    ("attention_prefill", "ri_attention_prefill"): [_P] * 8 + [_I] * 8 + [_F, _I, _P, _I, _F, _P, _I, _P, _P],
+    ("attention_prefill_tc", "ri_attention_prefill_tc"): [_P] * 8 + [_I] * 9 + [_F, _I, _P, _F, _P, _I, _I, _P, _P],
+    ("attention_prefill", "ri_attention_prefill"): [_P] * 8 + [_I] * 8 + [_F, _I, _P, _I, _F, _P, _I, _I, _P, _P],
 }
 DECODE_CHUNK = 128          # keys per partial result of the decode attention kernel
 MAX_FAST_HEAD_DIM = 256
@@ -344,17 +347,18 @@ def linear_heads(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
 def latent_prep(proj: torch.Tensor, q_col: int, dkv_col: int, qa: torch.Tensor, heads: int, dim: int, rot: int, rank: int,
                 gain: torch.Tensor, eps: float, rope_table: Optional[torch.Tensor], pool: Optional[torch.Tensor],
                 page_table: torch.Tensor, tok_seq: torch.Tensor, tok_pos: torch.Tensor, seq_slot: torch.Tensor,
-                write: bool = True) -> torch.Tensor:
+                write: bool = True, row: int = 0) -> torch.Tensor:
     """Latent attention between its projections and the attention over the cache.  ``proj`` [tokens, N] holds the
     heads' queries ([dim plain, rot to rotate] each) from column ``q_col`` and the down projection (rank + rot) from
     ``dkv_col``; ``qa`` [tokens, H, rank] the plain query parts already multiplied by the key up-projection.  Appends
     [RMS-normed latent, rotated shared key part] to ``pool`` [pages, 1, page_size, rank + rot] and returns the
-    query rows [tokens, H, rank + rot].  Rotation turns neighbouring pairs by ``rope_table`` [positions, rot/2, 2]."""
+    query rows [tokens, H, rank + rot].  ``row`` > rank + rot: both kinds of rows are that long, zeros at the end.  Rotation turns neighbouring pairs by ``rope_table`` [positions, rot/2, 2]."""
     _need(proj, "proj")
     tokens, ld = proj.shape
     _need(qa, "qa", proj.dtype, (tokens, heads, rank))
     _need(gain, "gain", torch.float32, (rank,))
     Dk = rank + rot
+    row = max(int(row), Dk)
     if q_col + heads * (dim + rot) > ld or dkv_col + Dk > ld:
         raise KernelError("latent_prep: the projection is narrower than its columns")
     rows = 0
@@ -372,18 +376,18 @@ def latent_prep(proj: torch.Tensor, q_col: int, dkv_col: int, qa: torch.Tensor, 
             raise KernelError("latent_prep: appending needs the cache pool")
         _need(pool, "pool", proj.dtype)
         pages, kvh, page_size, dk = pool.shape
-        if kvh != 1 or dk != Dk:
-            raise KernelError(f"latent_prep: pool {tuple(pool.shape)} does not fit one row of {Dk} per token")
+        if kvh != 1 or dk != row:
+            raise KernelError(f"latent_prep: pool {tuple(pool.shape)} does not fit one row of {row} per token")
     else:
         pages, page_size = 1, 1
     _need(page_table, "page_table", torch.int32)
     for t, n in ((tok_seq, "tok_seq"), (tok_pos, "tok_pos"), (seq_slot, "seq_slot")):
         _need(t, n, torch.int32)
-    qf = torch.empty((tokens, heads, Dk), dtype=proj.dtype, device=proj.device)
+    qf = torch.empty((tokens, heads, row), dtype=proj.dtype, device=proj.device)
     _call("latent_attention", "ri_latent_prep", proj.data_ptr(), ld, int(q_col), int(dkv_col), qa.data_ptr(), qf.data_ptr(),
           _ptr(pool) if write else None, page_table.data_ptr(), tok_seq.data_ptr(), tok_pos.data_ptr(), seq_slot.data_ptr(),
           gain.data_ptr(), float(eps), _ptr(rope_table), rows, tokens, heads, dim, rot, rank, page_table.shape[1], page_size,
-          pages, 1 if write else 0, _code(proj.dtype), error_flag(proj.device).data_ptr(), _stream())
+          pages, 1 if write else 0, row, _code(proj.dtype), error_flag(proj.device).data_ptr(), _stream())
     return qf
 
 
@@ -843,6 +847,59 @@ def rms_gains(resid: torch.Tensor, gains, eps: float, out_dtype: torch.dtype, te
     return outs
 
 
+def dyn_tanh(resid: torch.Tensor, alpha: torch.Tensor, gain: torch.Tensor, bias: torch.Tensor, out_dtype: torch.dtype,
+             delta: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
+             then: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """tanh(alpha x) * gain + bias for the float32 residual ``resid`` [n, dim], element by element in float32; ``alpha``
+    [1], ``gain`` and ``bias`` [dim] float32.  ``delta`` (compute dtype, same shape), ``rows`` and ``then`` as for
+    ``rmsnorm``: with ``delta`` the sum is taken first and written back unless ``rows`` is given."""
+    _need(resid, "resid", torch.float32)
+    n, dim = resid.shape
+    _need(alpha, "alpha", torch.float32, (1,))
+    _need(gain, "gain", torch.float32, (dim,))
+    _need(bias, "bias", torch.float32, (dim,))
+    if delta is not None:
+        _need(delta, "delta", out_dtype, (n, dim))
+    if rows is not None:
+        _need(rows, "rows", torch.int32)
+    n_out = n if rows is None else rows.numel()
+    out = torch.empty((n_out, dim), dtype=out_dtype, device=resid.device)
+    hint = _weight_hint(then, n_out) if out_dtype == torch.bfloat16 else None
+    _call("dyn_tanh", "ri_dyn_tanh", resid.data_ptr(), _ptr(delta), _ptr(rows), alpha.data_ptr(), gain.data_ptr(), bias.data_ptr(),
+          out.data_ptr(), n_out, dim, _code(out_dtype), _ptr(hint), hint.shape[0] if hint is not None else 0,
+          hint.shape[1] if hint is not None else 0, _stream())
+    return out
+
+
+def embed_dyn_tanh(ids: torch.Tensor, table: torch.Tensor, scale: float, alpha: torch.Tensor, gain: torch.Tensor,
+                   bias: torch.Tensor) -> torch.Tensor:
+    """float32 rows tanh(alpha * (table[ids] * scale)) * gain + bias."""
+    _need(ids, "ids", torch.int32)
+    _need(table, "table")
+    tokens, (vocab, dim) = ids.numel(), table.shape
+    _need(alpha, "alpha", torch.float32, (1,))
+    _need(gain, "gain", torch.float32, (dim,))
+    _need(bias, "bias", torch.float32, (dim,))
+    out = torch.empty((tokens, dim), dtype=torch.float32, device=table.device)
+    _call("dyn_tanh", "ri_embed_dyn_tanh", ids.data_ptr(), table.data_ptr(), float(scale), alpha.data_ptr(), gain.data_ptr(),
+          bias.data_ptr(), out.data_ptr(), tokens, dim, vocab, _code(table.dtype), error_flag(table.device).data_ptr(), _stream())
+    return out
+
+
+def pair_heads(x: torch.Tensor, lam: float, eps: float, gain: float, width: int, vdim: int) -> torch.Tensor:
+    """The two maps of differential attention put together: x [tokens, 2 H, Dp] holds head h's results a = x[:, 2h] and
+    b = x[:, 2h + 1] (``vdim`` true elements); o = a - lam b, then o / sqrt(mean(o^2) + eps) * gain, the mean over ``vdim``
+    elements, all in float32.  Returns [tokens, H, width] (``width`` >= vdim: zeros behind the true elements)."""
+    _need(x, "x")
+    tokens, two, Dp = x.shape
+    if two % 2 or not 0 < vdim <= min(width, Dp):
+        raise KernelError(f"pair_heads: {two} results of {Dp}, {vdim} elements in rows of {width}")
+    out = torch.empty((tokens, two // 2, width), dtype=x.dtype, device=x.device)
+    _call("pair_heads", "ri_pair_heads", x.data_ptr(), out.data_ptr(), float(lam), float(eps), float(gain), tokens, two // 2, Dp,
+          int(width), int(vdim), _code(x.dtype), _stream())
+    return out
+
+
 def embed_same(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor) -> None:
     """out[t] = table[ids[t]] in the table's own dtype; ``out`` [tokens, dim] may be a block of columns of a wider
     matrix (one half of the input of a product over two concatenated vectors)."""
@@ -862,7 +919,7 @@ def qkv_prep(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, heads: int,
              tok_seq: torch.Tensor, tok_pos: torch.Tensor, seq_slot: torch.Tensor, write_kv: bool = True,
              norm: str = "", q_gain: Optional[torch.Tensor] = None, k_gain: Optional[torch.Tensor] = None,
              norm_eps: float = 0.0, q_factor: Optional[torch.Tensor] = None, unit_v: bool = False,
-             Dv: int = 0) -> torch.Tensor:
+             Dv: int = 0, maps: int = 1) -> torch.Tensor:
     """Between the q/k/v product and the attention kernels: ``proj`` [tokens, N] holds the q heads from column ``q_col``,
     the k heads from ``k_col`` and the v heads from ``v_col`` (< 0: none, the values are the keys as cached), every head
     ``Dp`` columns wide with ``Dk`` true elements.  ``bias`` (float32, by column of the product) is added first; the first
@@ -876,7 +933,10 @@ def qkv_prep(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, heads: int,
     [H, Dp] and [KV, Dp]; eps ``norm_eps`` inside the root; the gains' padding columns are zero.
 
     ``q_factor`` [positions] (float32): the finished q heads are multiplied by their position's entry.  ``unit_v``: v heads
-    are divided by their root mean square over ``Dv`` elements (eps ``eps``).  ``kv_heads`` 0: only queries."""
+    are divided by their root mean square over ``Dv`` elements (eps ``eps``).  ``kv_heads`` 0: only queries.
+
+    ``maps`` > 1: a q head holds that many queries of Dk / maps elements side by side (a key head as many keys); the result
+    is [tokens, H * maps, Dp], every query in its own place of a row of zeros."""
     _need(proj, "proj")
     tokens, ld = proj.shape
     if norm not in ("", "head", "all"):
@@ -914,14 +974,14 @@ def qkv_prep(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, heads: int,
     _need(page_table, "page_table", torch.int32)
     for t, n in ((tok_seq, "tok_seq"), (tok_pos, "tok_pos"), (seq_slot, "seq_slot")):
         _need(t, n, torch.int32)
-    q = torch.empty((tokens, heads, Dp), dtype=proj.dtype, device=proj.device)
+    q = torch.empty((tokens, heads * maps, Dp), dtype=proj.dtype, device=proj.device)
     _call("qkv_prep", "ri_qkv_prep_norm", proj.data_ptr(), ld, int(q_col), int(k_col), int(v_col), _ptr(bias), q.data_ptr(),
           _ptr(k_pool) if write_kv else None, _ptr(v_pool) if write_kv and nv else None, page_table.data_ptr(),
           tok_seq.data_ptr(), tok_pos.data_ptr(), seq_slot.data_ptr(), _ptr(rope_table), rope_rows, int(rot),
           1 if pairs else 0, 1 if unit else 0, float(eps), _ptr(q_gain) if norm else None, _ptr(k_gain) if norm else None,
           {"": 0, "head": 1, "all": 2}[norm], float(norm_eps), _ptr(q_factor), 0 if q_factor is None else q_factor.numel(),
           1 if unit_v else 0, int(Dv or Dk), tokens, heads, kv_heads, Dp, Dk, page_table.shape[1], page_size,
-          pages, 1 if write_kv else 0, _code(proj.dtype), error_flag(proj.device).data_ptr(), _stream())
+          pages, 1 if write_kv else 0, int(maps), _code(proj.dtype), error_flag(proj.device).data_ptr(), _stream())
     return q
 
 
@@ -969,7 +1029,7 @@ def _bias(dist_bias: Optional[torch.Tensor], heads: int):
 def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_table: torch.Tensor,
               seq_slot: torch.Tensor, seq_start: torch.Tensor, seq_len: torch.Tensor, max_new: int, scale: float,
               window: int = 0, sink: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0,
-              dist_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+              dist_bias: Optional[torch.Tensor] = None, keep: int = 0) -> torch.Tensor:
     """Causal attention of the step's new tokens (q [tokens, H, Dh], sequences back to back as
     ``seq_start`` says) over the paged cache, which already holds their keys and values: float32 or
     bfloat16, any head size up to 512, any page size.  Every (token, head) is computed in one fixed
@@ -978,6 +1038,7 @@ def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_
     ``softcap`` > 0: score <- softcap * tanh(score / softcap) after the scale.
     ``dist_bias`` (float32, from ``pad_distance_bias``): added to the score after that, entry min(distance, n - 1) of the
     head's row of n.
+    ``keep`` > 0: beside a window a query also sees the sequence's first ``keep`` keys.
     ``v_pool`` may be ``k_pool`` itself (values that are the keys: latent attention)."""
     _need(q, "q")
     tokens, H, Dh = q.shape
@@ -995,7 +1056,7 @@ def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_
     _call("attention_rows", "ri_attention_rows", q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), out.data_ptr(),
           page_table.data_ptr(), seq_slot.data_ptr(), seq_start.data_ptr(), seq_len.data_ptr(), seqs, int(max_new),
           H, KV, Dh, page_table.shape[1], page_size, pages, float(scale), _mask(window, chunk), _sink(sink, H), _cap(softcap),
-          *_bias(dist_bias, H), _code(q.dtype), error_flag(q.device).data_ptr(), _stream())
+          *_bias(dist_bias, H), int(keep), _code(q.dtype), error_flag(q.device).data_ptr(), _stream())
     return out
 
 
@@ -1013,10 +1074,12 @@ def _decode_parts(head_dim: int, chunks: int) -> int:
 def attention_decode(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_table: torch.Tensor,
                      seq_slot: torch.Tensor, seq_len: torch.Tensor, scale: float, window: int,
                      max_len: int, sink: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0,
-                     dist_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     dist_bias: Optional[torch.Tensor] = None, keep: int = 0, pair=None) -> torch.Tensor:
     """Attention of one new token per sequence (q [seqs, H, Dh], bfloat16) over the
     paged cache, keys split into chunks of ``DECODE_CHUNK``; ``max_len`` bounds the
-    sequences' lengths after this step and sizes the scratch memory."""
+    sequences' lengths after this step and sizes the scratch memory.  ``keep`` as for ``attention``.
+    ``pair`` (lam, eps, gain, width, vdim): heads 2h and 2h + 1 are the two maps of differential attention, put together
+    as ``pair_heads`` does it, before anything is rounded; the result is then [seqs, H / 2, width]."""
     _need(q, "q", torch.bfloat16)
     seqs, H, Dh = q.shape
     pages, KV, page_size, dh = k_pool.shape
@@ -1033,24 +1096,27 @@ def attention_decode(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
     parts = _decode_parts(Dh, chunks)
     o_part = torch.empty((seqs, H, parts, Dh), dtype=torch.float32, device=q.device)
     ml_part = torch.empty((seqs, H, parts, 2), dtype=torch.float32, device=q.device)
-    out = torch.empty_like(q)
+    lam, eps, gain, width, vdim = pair or (0.0, 0.0, 0.0, 0, 0)
+    out = torch.empty_like(q) if pair is None else torch.empty((seqs, H // 2, width), dtype=q.dtype, device=q.device)
     _call("attention_decode", "ri_attention_decode_cap", q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(),
           out.data_ptr(), o_part.data_ptr(), ml_part.data_ptr(), page_table.data_ptr(), seq_slot.data_ptr(),
           seq_len.data_ptr(), seqs, H, KV, Dh, page_table.shape[1], page_size, pages, chunks, float(scale),
-          _mask(window, chunk), _sink(sink, H), _cap(softcap), *_bias(dist_bias, H), error_flag(q.device).data_ptr(), _stream(),
-          defines={"RI_HEAD_DIM": Dh})
+          _mask(window, chunk), _sink(sink, H), _cap(softcap), *_bias(dist_bias, H), int(keep), int(width), int(vdim), float(lam),
+          float(eps), float(gain), error_flag(q.device).data_ptr(), _stream(), defines={"RI_HEAD_DIM": Dh})
     return out
 
 
 def attention_prefill(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_table: torch.Tensor,
                       seq_slot: torch.Tensor, seq_start: torch.Tensor, seq_len: torch.Tensor, max_new: int,
                       scale: float, window: int, sink: Optional[torch.Tensor] = None, v_dims: int = 0,
-                      chunk: int = 0, softcap: float = 0.0, dist_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      chunk: int = 0, softcap: float = 0.0, dist_bias: Optional[torch.Tensor] = None,
+                      keep: int = 0) -> torch.Tensor:
     """Attention of the step's new tokens (q [tokens, H, Dh], bfloat16, sequences back
     to back as ``seq_start`` says) over the paged cache, which already holds their keys
     and values; ``max_new`` is the most tokens one sequence brings.  ``v_pool`` may be ``k_pool``
     itself (values that are the keys): the mma.sync kernel then reads each tile once; ``v_dims`` > 0
-    says that only that many leading elements of the result are wanted (the rest may be zeros)."""
+    says that only that many leading elements of the result are wanted (the rest may be zeros).  ``keep`` as for
+    ``attention``."""
     _need(q, "q", torch.bfloat16)
     tokens, H, Dh = q.shape
     pages, KV, page_size, dh = k_pool.shape
@@ -1071,13 +1137,13 @@ def attention_prefill(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tenso
         _call("attention_prefill_tc", "ri_attention_prefill_tc", q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(),
               out.data_ptr(), page_table.data_ptr(), seq_slot.data_ptr(), seq_start.data_ptr(), seq_len.data_ptr(),
               q.shape[0], seqs, int(max_new), H, KV, Dh, page_table.shape[1], page_size, pages, float(scale),
-              _mask(window, chunk), _sink(sink, H), _cap(softcap), *_bias(dist_bias, H), error_flag(q.device).data_ptr(), _stream(),
-              defines={"RI_HEAD_DIM": Dh})
+              _mask(window, chunk), _sink(sink, H), _cap(softcap), *_bias(dist_bias, H), int(keep), error_flag(q.device).data_ptr(),
+              _stream(), defines={"RI_HEAD_DIM": Dh})
         return out
     _call("attention_prefill", "ri_attention_prefill", q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(),
           out.data_ptr(), page_table.data_ptr(), seq_slot.data_ptr(), seq_start.data_ptr(), seq_len.data_ptr(),
           seqs, int(max_new), H, KV, Dh, page_table.shape[1], page_size, pages, float(scale), _mask(window, chunk),
-          _sink(sink, H), int(v_dims), _cap(softcap), *_bias(dist_bias, H), error_flag(q.device).data_ptr(), _stream(), defines={"RI_HEAD_DIM": Dh})
+          _sink(sink, H), int(v_dims), _cap(softcap), *_bias(dist_bias, H), int(keep), error_flag(q.device).data_ptr(), _stream(), defines={"RI_HEAD_DIM": Dh})
     return out
 
 
@@ -1317,11 +1383,12 @@ def linear_gated(x: torch.Tensor, w_gate_up: torch.Tensor, block: int, kind: str
     return gated_act(linear(x, w_gate_up), kind, block, limit, alpha)
 
 
-MOE_SCORES = {"softmax": 0, "sigmoid": 1}
+MOE_SCORES = {"softmax": 0, "sigmoid": 1, "logits": 2}
 
 
-def moe_route(x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor, top: int, score: str = "softmax",
-              groups: int = 1, keep: int = 1, group_top: int = 2, scale: float = 1.0, renormalize: bool = True):
+def moe_route(x: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], top: int, score: str = "softmax",
+              groups: int = 1, keep: int = 1, group_top: int = 2, scale: float = 1.0, renormalize: bool = True,
+              bias: Optional[torch.Tensor] = None):
     """Per token the ``top`` router outputs with the largest softmax(router x) + correction (ties: the lower index),
     and as weights their softmax scores divided by their sum (+ 1e-20).  ``router`` [N, D] and ``correction`` [N]
     float32.  Returns (int32 [tokens, top], float32 [tokens, top]).
@@ -1329,21 +1396,27 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor, t
     ``score`` "sigmoid": the scores are the sigmoid of every output on its own.  ``groups`` > 1: the outputs form that
     many equal runs of neighbours, a run's score is the sum of its ``group_top`` largest choice scores, and only outputs
     of the ``keep`` best runs can be chosen.  The weights are multiplied by ``scale``; ``renormalize`` False leaves out
-    the division by their sum."""
+    the division by their sum.  ``score`` "logits": the choice is by the router's outputs themselves (``correction``
+    None), and the weights are the softmax over the chosen outputs alone (times ``scale``).  ``bias`` [N] (float32) is added
+    to the outputs first."""
     _need(x, "x")
     tokens, D = x.shape
     _need(router, "router", torch.float32)
     N = router.shape[0]
     if router.shape[1] != D:
         raise KernelError(f"moe_route: router {tuple(router.shape)} does not fit rows of {D}")
-    _need(correction, "correction", torch.float32, (N,))
+    if (correction is None) != (score == "logits"):
+        raise KernelError(f"moe_route: score {score!r} goes {'without' if score == 'logits' else 'with'} a correction")
+    for t, name in ((correction, "correction"), (bias, "bias")):
+        if t is not None:
+            _need(t, name, torch.float32, (N,))
     idx = torch.empty((tokens, top), dtype=torch.int32, device=x.device)
     weight = torch.empty((tokens, top), dtype=torch.float32, device=x.device)
     if score not in MOE_SCORES:
         raise KernelError(f"moe_route: score {score!r} (known: {', '.join(sorted(MOE_SCORES))})")
-    _call("moe", "ri_moe_route_rule", x.data_ptr(), router.data_ptr(), correction.data_ptr(), idx.data_ptr(), weight.data_ptr(),
+    _call("moe", "ri_moe_route_rule", x.data_ptr(), router.data_ptr(), _ptr(correction), idx.data_ptr(), weight.data_ptr(),
           tokens, D, N, int(top), MOE_SCORES[score], int(groups), int(keep), int(group_top), float(scale),
-          1 if renormalize else 0, _code(x.dtype), _stream())
+          1 if renormalize else 0, _ptr(bias), _code(x.dtype), _stream())
     return idx, weight
 
 

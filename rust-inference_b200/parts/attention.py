@@ -21,11 +21,18 @@ the mixer's input (or one gate per head), stacked into the q/k/v product; a norm
 before the rotation that runs over the whole projection of a token instead of over each head; values divided by
 their root mean square before they are cached; a factor on the queries that grows with the position; a learned
 bias on the scores by distance (``parts/distance.py``); no keys and values of its own (the layer reads the cache
-entry that another layer writes).  A record
+entry that another layer writes); kept first tokens beside a window.  A record
 that uses any of them (or a per-head norm together with values of another size) runs the
 "extended" order of work: one product for q, k, (v), (gate); ``ops.qkv_prep`` (bias, rotation,
 unit norm, append); attention; gate; output projection.  Heads are then always padded to a
 multiple of 16 elements, so that the tensor-core kernels take every size.
+
+Differential attention (``maps`` 2): a key head's two keys stand side by side in the cache as ONE key of twice the size, over
+one value, so nothing is stored twice.  A query head becomes two query heads of that size, each with its own query in its
+place and zeros in the other's (``ops.qkv_prep``): a zero times a key element adds exactly 0, so its score against the
+whole key is its map's score, and the attention kernels run 2 H heads over the G key heads as they are.  The two maps of a
+head are neighbours; they are put together in float32 by the merge of the decode kernel's partial results, or behind the
+other attention kernels (``ops.pair_heads``): difference, norm over the value's elements, constant factor.
 """
 from __future__ import annotations
 
@@ -79,7 +86,19 @@ class Attention(Mixer):
         self.bias_rows = int(getattr(spec, "bias_rows", 0) or 0)
         self.own_kv = bool(getattr(spec, "own_kv", True))
         self.q_factor = self.dist_bias = None
-        self.extended = bool(self.bias_of or self.keys_are_values or self.unit_rms or self.softcap or self.gated
+        self.maps = int(getattr(spec, "maps", 1))
+        self.keep = int(getattr(spec, "keep_first", 0)) if spec.window else 0
+        if self.maps not in (1, 2):
+            raise ValueError(f"{self.maps} maps per head: 1 or 2 (differential attention)")
+        if self.maps == 2:
+            if self.rot or spec.qk_norm is not None or self.unit_rms or self.bias_of or self.keys_are_values or self.gated \
+                    or self.bias_rows or spec.sink:
+                raise ValueError("differential attention is built without a rotation, norms of queries and keys, biases, gates, "
+                                 "a distance bias or a sink")
+            self.Dk = 2 * spec.head_dim
+            self.Dv = spec.v_head_dim or spec.head_dim
+        self.lam = 0.0
+        self.extended = bool(self.maps > 1 or self.bias_of or self.keys_are_values or self.unit_rms or self.softcap or self.gated
                              or self.unit_values or self.temperature or self.bias_rows or not self.own_kv
                              or self.norm_span == "all" or (self.norm_span and self.Dp != self.Dk))
         if self.extended:
@@ -91,11 +110,15 @@ class Attention(Mixer):
                 raise ValueError("values that are the keys are cached as the keys are, without a norm of their own")
             self.Dp = -(-max(self.Dk, self.Dv) // 16) * 16
             self.bias = None
+        # elements of a head's row in front of the output matrix
+        self.Do = self.Dp if self.maps == 1 else -(-self.Dv // 16) * 16
 
     @classmethod
     def param_infos(cls, spec):
         D, H, KV, Dh = spec.hidden_size, spec.num_heads, spec.num_kv_heads, spec.head_dim
         Dv = spec.v_head_dim or Dh
+        maps = getattr(spec, "maps", 1)
+        Dh = maps * Dh                                 # of a query head and a key head
         q, k, v, o, sink = spec.names
         infos = {q: ParamInfo((H * Dh, D)), k: ParamInfo((KV * Dh, D)), v: ParamInfo((KV * Dv, D)), o: ParamInfo((D, H * Dv))}
         if getattr(spec, "values", "own") == "keys" or not getattr(spec, "own_kv", True):
@@ -118,6 +141,9 @@ class Attention(Mixer):
                 infos[kn] = ParamInfo((KV * Dh if whole else Dh,), "gain")
         if spec.sink:
             infos[sink] = ParamInfo((H,), "vector")
+        if maps == 2:
+            for name in spec.pair_names:
+                infos[name] = ParamInfo((spec.head_dim,), "vector")
         return infos
 
     def load(self, tensors):
@@ -163,10 +189,10 @@ class Attention(Mixer):
                         bias[col:col + heads * Dp].view(heads, Dp)[:, :size] = tensors[name + s.bias_suffix].float().view(heads, size)
                 self.bias = bias
         wo = tensors[o]
-        if self.Dv != Dp:
-            padded = wo.new_zeros((D, s.num_heads, Dp))
+        if self.Dv != self.Do:
+            padded = wo.new_zeros((D, s.num_heads, self.Do))
             padded[:, :, :self.Dv] = wo.view(D, s.num_heads, self.Dv)
-            wo = padded.view(D, s.num_heads * Dp)
+            wo = padded.view(D, s.num_heads * self.Do)
         self.o = wo.contiguous()
         if s.qk_norm is not None:
             qn, kn = getattr(s, "qk_norm_names", ("q_norm.weight", "k_norm.weight"))
@@ -185,6 +211,9 @@ class Attention(Mixer):
                 self.k_gain = padded(self.k_gain, s.num_kv_heads) if own else None
         if s.sink:
             self.sink = tensors[sink]
+        if self.maps == 2:
+            q1, k1, q2, k2 = (tensors[n].double() for n in s.pair_names)
+            self.lam = float(torch.exp((q1 * k1).sum()) - torch.exp((q2 * k2).sum())) + float(s.pair_diff)
         if self.bias_rows:
             self.dist_bias = ops.pad_distance_bias(spread_over_distances(tensors[s.bias_name], s.bias_far))
 
@@ -197,7 +226,7 @@ class Attention(Mixer):
     def cache_request(self):
         s = self.spec
         return CacheRequest(kv_heads=s.num_kv_heads, head_dim=self.Dp, window=s.window, chunk=s.chunk,
-                            shared_kv=self.keys_are_values)
+                            shared_kv=self.keys_are_values, keep_first=self.keep)
 
     def prepare(self, max_positions):
         self.position.prepare(max_positions)
@@ -223,26 +252,30 @@ class Attention(Mixer):
                              self.unit_rms, s.unit_eps, cache.k_pool, cache.v_pool, cache.page_table, ctx.tok_seq,
                              ctx.tok_pos, ctx.seq_slot, write_kv=cache.writes, norm=self.norm_span, q_gain=self.q_gain,
                              k_gain=self.k_gain, norm_eps=s.qk_norm.eps if s.qk_norm is not None else 0.0,
-                             q_factor=self.q_factor, unit_v=self.unit_values, Dv=self.Dv)
+                             q_factor=self.q_factor, unit_v=self.unit_values, Dv=self.Dv, maps=self.maps)
         fast = ops.fast_attention_supported(q.dtype, Dp, cache.page_size)
+        pair = (self.lam, s.pair_eps, 1.0 - s.pair_diff, self.Do, self.Dv) if self.maps == 2 else None
         with section("attention"):
             if fast and ctx.decode_only:
                 out = ops.attention_decode(q, cache.k_pool, cache.v_pool, cache.page_table, ctx.seq_slot, ctx.seq_len,
                                            self.scale, s.window, ctx.len_bucket, softcap=self.softcap,
-                                           dist_bias=self.dist_bias)
+                                           dist_bias=self.dist_bias, keep=self.keep, pair=pair)
             elif fast:
                 out = ops.attention_prefill(q, cache.k_pool, cache.v_pool, cache.page_table, ctx.seq_slot,
                                             ctx.seq_start, ctx.seq_len, ctx.max_new, self.scale, s.window,
-                                            softcap=self.softcap, dist_bias=self.dist_bias)
+                                            softcap=self.softcap, dist_bias=self.dist_bias, keep=self.keep)
             else:
                 out = ops.attention(q, cache.k_pool, cache.v_pool, cache.page_table, ctx.seq_slot, ctx.seq_start,
                                     ctx.seq_len, ctx.max_new, self.scale, s.window, softcap=self.softcap,
-                                    dist_bias=self.dist_bias)
+                                    dist_bias=self.dist_bias, keep=self.keep)
+        if pair is not None and not (fast and ctx.decode_only):
+            with section("attn pairs"):
+                out = ops.pair_heads(out, *pair)
         if self.gated:
             with section("attn gate"):
                 ops.gate_heads(out, proj[:, self.g_col:self.g_col + (H if self.gated == "head" else H * Dp)], "sigmoid")
         with section("attn o proj"):
-            return ops.linear(out.view(T, H * Dp), self.o)
+            return ops.linear(out.view(T, H * self.Do), self.o)
 
     def __call__(self, x, ctx, cache):
         if self.extended:
@@ -278,13 +311,14 @@ class Attention(Mixer):
         with section("attention"):
             if fast and ctx.decode_only:
                 out = ops.attention_decode(q, cache.k_pool, cache.v_pool, cache.page_table, ctx.seq_slot, ctx.seq_len,
-                                           self.scale, s.window, ctx.len_bucket, sink=self.sink, chunk=s.chunk)
+                                           self.scale, s.window, ctx.len_bucket, sink=self.sink, chunk=s.chunk,
+                                           keep=self.keep)
             elif fast:
                 out = ops.attention_prefill(q, cache.k_pool, cache.v_pool, cache.page_table, ctx.seq_slot,
                                             ctx.seq_start, ctx.seq_len, ctx.max_new, self.scale, s.window, sink=self.sink,
-                                            chunk=s.chunk)
+                                            chunk=s.chunk, keep=self.keep)
             else:
                 out = ops.attention(q, cache.k_pool, cache.v_pool, cache.page_table, ctx.seq_slot, ctx.seq_start,
-                                    ctx.seq_len, ctx.max_new, self.scale, s.window, sink=self.sink, chunk=s.chunk)
+                                    ctx.seq_len, ctx.max_new, self.scale, s.window, sink=self.sink, chunk=s.chunk, keep=self.keep)
         with section("attn o proj"):
             return ops.linear(out.view(x.shape[0], s.num_heads * self.Dp), self.o)

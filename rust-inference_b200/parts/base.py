@@ -24,7 +24,7 @@ FeedForward     ``__call__(x, ctx) -> y``
 """
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Dict, Optional
 
 import torch
@@ -82,7 +82,8 @@ class CacheRequest:
     Keys and values: ``kv_heads`` x ``head_dim`` per token (0 for none), all of
     them (``window`` 0) or the last ``window``; ``chunk`` > 0 instead of a window: the
     keys of the query's own chunk of that many positions, counted from the sequence's
-    start.  ``shared_kv``: the values are the keys (a latent that serves as both), so
+    start.  ``keep_first``: beside the window, the sequence's first tokens, which every query
+    sees however far behind they are.  ``shared_kv``: the values are the keys (a latent that serves as both), so
     one pool is kept and handed out as both.
     Fixed-size state: ``state_shape`` per sequence (empty for none), zeroed when a
     slot is given out; ``more_state``: further such tensors as (shape, dtype) pairs,
@@ -95,6 +96,24 @@ class CacheRequest:
     shared_kv: bool = False
     chunk: int = 0
     more_state: tuple = ()
+    keep_first: int = 0
+
+    @property
+    def kept(self) -> int:
+        """First tokens that stay stored beside a window (0 where everything, or a chunk, stays anyway)."""
+        if self.keep_first and self.chunk:
+            raise ValueError("kept first tokens go with a window, not with a chunked mask")
+        return self.keep_first if self.window else 0
+
+    def for_readers(self, others) -> "CacheRequest":
+        """This request of a writing layer, widened so that layers that read the same entry through masks of their own
+        (``others``: their requests) find every key they see."""
+        masks = [(r.window, r.chunk, r.kept) for r in (self, *others)]
+        if len(set(masks)) == 1:
+            return self
+        if all(w > 0 for w, _, _ in masks):
+            return replace(self, window=max(w for w, _, _ in masks), chunk=0, keep_first=max(k for _, _, k in masks))
+        return replace(self, window=0, chunk=0, keep_first=0)
 
     @property
     def mask(self) -> int:

@@ -45,12 +45,16 @@ class BlockBase:
 class PreNormBlock(BlockBase):
     @classmethod
     def slots(cls, spec):
-        return (("mixer_norm", "norm", spec.mixer_norm), ("mixer", "mixer", spec.mixer),
-                ("ffn_norm", "norm", spec.ffn_norm), ("ffn", "ffn", spec.ffn))
+        out = (("mixer_norm", "norm", spec.mixer_norm), ("mixer", "mixer", spec.mixer))
+        if spec.ffn is not None:
+            out += (("ffn_norm", "norm", spec.ffn_norm), ("ffn", "ffn", spec.ffn))
+        return out
 
     def __call__(self, resid, delta, ctx, cache):
         x = norm_before(self.mixer_norm, resid, delta, self.mixer)
         a = self.mixer(x, ctx, cache)
+        if self.spec.ffn is None:
+            return resid, a
         x = norm_before(self.ffn_norm, resid, a, self.ffn)
         return resid, self.ffn(x, ctx)
 

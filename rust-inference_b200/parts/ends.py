@@ -1,7 +1,8 @@
 """The two ends of the model: token ids in, logits out.
 
 ``embedding``: h[t] = table[ids[t]] as float32 rows of the residual stream (times the record's
-``scale``, 1 by default, and repeated ``copies`` times for a residual kept as several streams); an id
+``scale``, 1 by default, and repeated ``copies`` times for a residual kept as several streams), passed through a
+norm if the record names one; an id
 outside the table is reported through the error word (thanhauco/rust-inference
 src/ops/embedding.rs:10-42).
 
@@ -23,23 +24,37 @@ from __future__ import annotations
 import torch
 
 from .. import ops
-from .base import CacheRequest, Part
-from .registry import ParamInfo, register_embedding, register_head
+from .base import BuildEnv, CacheRequest, Part
+from .registry import ParamInfo, build_part, part_class, register_embedding, register_head
 
 
 @register_embedding("embedding")
 class TokenEmbedding(Part):
     graph_safe = True
 
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.norm = None
+        if getattr(spec, "norm", None) is not None:
+            if getattr(spec, "copies", 1) != 1:
+                raise ValueError("an embedding whose rows are normed has one stream")
+            # the normed rows are the residual: float32 whatever the compute dtype
+            self.norm = build_part("norm", spec.norm, BuildEnv(torch.float32, env.device))
+
     @classmethod
     def param_infos(cls, spec):
         infos = {"weight": ParamInfo((spec.vocab_size, spec.hidden_size), "matrix")}
+        if getattr(spec, "norm", None) is not None:
+            for local, info in part_class("norm", spec.norm).param_infos(spec.norm).items():
+                infos["norm" + local] = info
         if getattr(spec, "side_width", 0):
             infos[spec.side_name] = ParamInfo((spec.vocab_size, spec.side_width), "matrix")
         return infos
 
     def load(self, tensors):
         self.table = tensors["weight"]
+        if self.norm is not None:
+            self.norm.load({k[len("norm"):]: v for k, v in tensors.items() if k.startswith("norm")})
         # a second table of token rows: the layers' token-fed sublayers read their columns of it
         self.side = tensors[self.spec.side_name] if getattr(self.spec, "side_width", 0) else None
 
@@ -47,6 +62,11 @@ class TokenEmbedding(Part):
         return self.table.numel() * self.table.element_size()
 
     def __call__(self, ids, ctx=None):
+        if self.norm is not None:
+            scale = getattr(self.spec, "scale", 1.0)
+            if hasattr(self.norm, "of_rows"):
+                return self.norm.of_rows(ids, self.table, scale)
+            return self.norm(ops.embed(ids, self.table, scale))
         return ops.embed(ids, self.table, getattr(self.spec, "scale", 1.0), getattr(self.spec, "copies", 1))
 
 

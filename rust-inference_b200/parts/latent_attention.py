@@ -9,7 +9,8 @@ With h the mixer's input, per token:
     score  = (q_plain . Wuk_h c + rotate(q_rot) . r) * scale,  causal, the last ``window`` keys
     softmax, with exp(sink_h) in the denominator if the record says so
     out    = Wo concat_h(gate_h * sum_j p_j v_hj),  gate = sigmoid(Wg h) per head or per element
-Only [c, r] is cached: one row of kv_rank + rot_dim per token.
+Only [c, r] is cached: one row of kv_rank + rot_dim per token, with zeros up to a multiple of 16 elements (the sizes that
+the tensor-core attention kernels take; in float32 too, where any size would do).
 
 Order of work here: the three projections of h are one product with the stacked matrix; the key up-projection
 is folded into the query (qa_h = Wuk_h^T q_plain: a product per head), so that the score against a cached row is
@@ -45,6 +46,7 @@ class LatentAttention(Mixer):
         if spec.rot_dim and not getattr(self.position, "pairs", False):
             raise ValueError(f"latent attention turns neighbouring pairs; position kind {spec.position.kind!r} does not")
         self.sink = None
+        self.row = -(-(spec.kv_rank + spec.rot_dim) // 16) * 16
 
     @classmethod
     def gate_rows(cls, spec) -> int:
@@ -84,14 +86,14 @@ class LatentAttention(Mixer):
 
     def cache_request(self):
         s = self.spec
-        return CacheRequest(kv_heads=1, head_dim=s.kv_rank + s.rot_dim, window=s.window, shared_kv=True)
+        return CacheRequest(kv_heads=1, head_dim=self.row, window=s.window, shared_kv=True)
 
     def prepare(self, max_positions):
         self.position.prepare(max_positions)
 
     def __call__(self, x, ctx, cache):
         s = self.spec
-        T, H, Dk = x.shape[0], s.num_heads, s.kv_rank + s.rot_dim
+        T, H = x.shape[0], s.num_heads
         with section("latent q/dkv/gate proj"):
             proj = ops.linear(x, self.proj)
         with section("latent key fold"):
@@ -100,9 +102,9 @@ class LatentAttention(Mixer):
         with section("latent norm/rope/append"):
             qf = ops.latent_prep(proj, self.q_col, self.dkv_col, qa, H, s.dim, s.rot_dim, s.kv_rank, self.latent_gain, s.eps,
                                  self.position.fused_table(), cache.k_pool, cache.page_table, ctx.tok_seq, ctx.tok_pos,
-                                 ctx.seq_slot, write=cache.writes)
+                                 ctx.seq_slot, write=cache.writes, row=self.row)
         pool = cache.k_pool
-        fast = ops.fast_attention_supported(qf.dtype, Dk, cache.page_size)
+        fast = ops.fast_attention_supported(qf.dtype, self.row, cache.page_size)
         with section("attention"):
             if fast and ctx.decode_only:
                 lat = ops.attention_decode(qf, pool, pool, cache.page_table, ctx.seq_slot, ctx.seq_len, s.scale, s.window,

@@ -169,8 +169,8 @@ class PassMix(Part):
     def bind(self, embedding) -> None:
         """The model's embedding part: rows of its ``table`` are the second half of the product's input."""
         if getattr(embedding.spec, "kind", "") != "embedding" or float(getattr(embedding.spec, "scale", 1.0)) != 1.0 \
-                or getattr(embedding.spec, "copies", 1) != 1:
-            raise ValueError("a pass that mixes the embedding's output in needs the plain embedding (no factor, one stream)")
+                or getattr(embedding.spec, "copies", 1) != 1 or getattr(embedding.spec, "norm", None) is not None:
+            raise ValueError("a pass that mixes the embedding's output in needs the plain embedding (no factor, no norm, one stream)")
         self.embedding = embedding
 
     def enter(self, resid, delta, t: int, ids):
@@ -223,7 +223,8 @@ class PassEntry(Part):
 
     def bind(self, embedding) -> None:
         """The model's embedding part: its ``table`` and the factor of its record are what is added again."""
-        if self.spec.readd_embedding and getattr(embedding.spec, "kind", "") != "embedding":
+        if self.spec.readd_embedding and (getattr(embedding.spec, "kind", "") != "embedding"
+                                          or getattr(embedding.spec, "norm", None) is not None):
             raise ValueError("a pass that adds the embedding's output again needs the plain (scaled) embedding")
         self.embedding = embedding
 

@@ -4,7 +4,8 @@
     w_j = s[choice_j] / (sum_j s[choice_j] + 1e-20)
 Options of the record: s = sigmoid(z) element by element; a choice only among the experts of the best groups of
 neighbouring experts (a group's score: the sum of its largest choice scores); weights that are not divided by their
-sum; a constant factor on the weights; no router at all, but an integer table that names every token id's experts,
+sum; a constant factor on the weights; a bias on the router's outputs; a choice by the outputs z themselves with the softmax
+over the chosen ones as weights, without a correction (``score`` "logits"); no router at all, but an integer table that names every token id's experts,
 each with weight 1 / top (``route`` "table").
     y = sum_j w_j expert_{choice_j}(h)  (+ shared(h))
 The router's last ``identity`` outputs stand for experts that return h itself and have no tensors.  The experts are
@@ -58,7 +59,11 @@ class MixtureOfExperts(FeedForward):
         if getattr(spec, "route", "scores") == "table":
             infos = {spec.table_name: ParamInfo((spec.table_rows, spec.top), "table", below=spec.experts)}
         else:
-            infos = {"router": ParamInfo((N, D), "vector"), "correction": ParamInfo((N,), "vector")}
+            infos = {"router": ParamInfo((N, D), "vector")}
+            if getattr(spec, "score", "softmax") != "logits":
+                infos["correction"] = ParamInfo((N,), "vector")
+            if getattr(spec, "router_bias", ""):
+                infos[spec.router_bias] = ParamInfo((N,), "vector")
         for e in range(spec.experts):
             infos[f"e{e}.gate"], infos[f"e{e}.up"] = ParamInfo((I, D)), ParamInfo((I, D))
             infos[f"e{e}.down"] = ParamInfo((D, I))
@@ -72,7 +77,8 @@ class MixtureOfExperts(FeedForward):
         if self.by_table:
             self.table = tensors[self.spec.table_name].contiguous()
         else:
-            self.router, self.correction = tensors["router"], tensors["correction"]
+            self.router, self.correction = tensors["router"], tensors.get("correction")
+            self.router_bias = tensors.get(getattr(self.spec, "router_bias", "") or "-")
         # per expert [gate rows; up rows], all experts stacked
         self.gate_up = torch.stack([torch.cat([tensors[f"e{e}.gate"], tensors[f"e{e}.up"]], dim=0) for e in range(E)]).contiguous()
         self.down = torch.stack([tensors[f"e{e}.down"] for e in range(E)]).contiguous()
@@ -97,7 +103,7 @@ class MixtureOfExperts(FeedForward):
             else:
                 idx, weight = ops.moe_route(x, self.router, self.correction, s.top, getattr(s, "score", "softmax"),
                                             getattr(s, "groups", 1), getattr(s, "group_keep", 1), getattr(s, "group_top", 2),
-                                            getattr(s, "route_scale", 1.0), getattr(s, "renormalize", True))
+                                            getattr(s, "route_scale", 1.0), getattr(s, "renormalize", True), bias=self.router_bias)
                 plan = ops.moe_plan(idx, s.experts, wide)
         with section("moe experts"):
             gu = ops.moe_grouped_linear(x, self.gate_up, plan, T * s.top, gather_div=s.top)

@@ -7,7 +7,9 @@ LayerNorm: y = (x - mean) / sqrt(var + eps) * gain (+ bias, where the record nam
 the mean squared deviation, float32.  It reads a residual of one or several streams ([tokens, dim] or
 [tokens, streams, dim]): the pending output joins the streams by its connection's weights
 (:class:`~.base.Pending`) and the row that is normed is the streams' weighted sum (``read``;
-absent: their plain sum), all in the same kernel."""
+absent: their plain sum), all in the same kernel.
+
+Dynamic Tanh: tanh(alpha x) * gain + bias, element by element, float32."""
 from __future__ import annotations
 
 import torch
@@ -142,3 +144,38 @@ class NoNorm(Norm):
         with section("residual"):
             ops.rms_gains(resid, (), 0.0, self.env.dtype, terms=terms, entry=entry, post=post, out=out, then=then)
         return out
+
+
+@register_norm("dyn_tanh")
+class DynTanh(Norm):
+    """tanh(alpha x) * gain + bias of the (single-stream) residual, element by element (no mean, no variance).  The
+    sublayer's output that is pending joins in the same pass, in float32; anything more than one output without a factor
+    joins in a pass of its own in front (the kernel of ``rms_gains`` without a norm)."""
+    graph_safe = True
+    takes_hint = True
+
+    @classmethod
+    def param_infos(cls, spec):
+        return {spec.weight_name: ParamInfo((spec.size,), "gain"), spec.bias_name: ParamInfo((spec.size,), "vector"),
+                spec.alpha_name: ParamInfo((), "gain")}
+
+    def load(self, tensors):
+        s = self.spec
+        self.gain, self.bias = tensors[s.weight_name], tensors[s.bias_name]
+        self.alpha = tensors[s.alpha_name].reshape(1).contiguous()
+
+    def weight_bytes(self):
+        return 4 * (self.gain.numel() + self.bias.numel() + 1)
+
+    def __call__(self, resid, delta=None, rows=None, then=None):
+        resid, terms, entry, post = _single_stream(resid, delta)
+        with section("dyn_tanh"):
+            if len(terms) > 1 or entry is not None or post is not None or (terms and terms[0][1] is not None):
+                ops.rms_gains(resid, (), 0.0, self.env.dtype, terms=terms, entry=entry, post=post)
+                terms = []
+            return ops.dyn_tanh(resid, self.alpha, self.gain, self.bias, self.env.dtype, delta=terms[0][0] if terms else None,
+                                rows=rows, then=then)
+
+    def of_rows(self, ids, table, scale):
+        """The norm of the rows table[ids] * scale, in float32 (an embedding whose rows are normed), in one pass."""
+        return ops.embed_dyn_tanh(ids, table, scale, self.alpha, self.gain, self.bias)

@@ -73,7 +73,7 @@ class ParallelMixer(Mixer):
             return None
         first = states[0] if states else ((), None)
         return CacheRequest(kv_heads=kv.kv_heads if kv else 0, head_dim=kv.head_dim if kv else 0,
-                            window=kv.window if kv else 0, chunk=kv.chunk if kv else 0,
+                            window=kv.window if kv else 0, chunk=kv.chunk if kv else 0, keep_first=kv.keep_first if kv else 0,
                             shared_kv=kv.shared_kv if kv else False, state_shape=first[0],
                             state_dtype=first[1] if states else CacheRequest().state_dtype, more_state=tuple(states[1:]))
 

@@ -18,7 +18,8 @@ __all__ = ["embed", "rmsnorm", "add_rows", "silu_mul", "linear_swiglu", "linear"
            "sample", "mark_seen", "stream_norm", "activation", "gate_heads", "linear_heads", "latent_prep", "gla_recurrent",
            "head_norm_gate", "linear_act", "scale_", "embed_pair_hash", "short_conv", "delta_rule_recurrent", "gated_act",
            "linear_gated", "moe_route", "moe_plan", "moe_grouped_linear", "moe_combine", "rms_gains", "qkv_prep", "softcap_",
-           "embed_same", "mlstm_gates", "scalar_decay_recurrent", "mlstm_head_norm_gate", "moe_plan_table", "linear_act_rows"]
+           "embed_same", "mlstm_gates", "scalar_decay_recurrent", "mlstm_head_norm_gate", "moe_plan_table", "linear_act_rows",
+           "dyn_tanh", "embed_dyn_tanh", "pair_heads"]
 
 
 def embed(ids, table, scale=1.0, copies=1):
@@ -84,7 +85,7 @@ def linear_heads(x, w):
 
 
 def latent_prep(proj, q_col, dkv_col, qa, heads, dim, rot, rank, gain, eps, rope_table, pool, page_table, tok_seq, tok_pos,
-                seq_slot, write=True):
+                seq_slot, write=True, row=0):
     T = proj.shape[0]
     p = proj.float()
 
@@ -98,7 +99,8 @@ def latent_prep(proj, q_col, dkv_col, qa, heads, dim, rot, rank, gain, eps, rope
     down = p[:, dkv_col:dkv_col + rank + rot]
     c = down[:, :rank]
     c = c / torch.sqrt((c * c).mean(-1, keepdim=True) + eps) * gain
-    row = torch.cat([c, turn(down[:, rank:]) if rot else down[:, rank:]], dim=-1)
+    pad = max(row - rank - rot, 0)
+    row = torch.cat([c, turn(down[:, rank:]) if rot else down[:, rank:], torch.zeros(T, pad)], dim=-1)
     if write:
         P = pool.shape[2]
         for t in range(T):
@@ -108,7 +110,7 @@ def latent_prep(proj, q_col, dkv_col, qa, heads, dim, rot, rank, gain, eps, rope
             pool[page, 0, pos % P, :] = row[t].to(pool.dtype)
     q = p[:, q_col:q_col + heads * (dim + rot)].view(T, heads, dim + rot)
     qr = turn(q[..., dim:]) if rot else q[..., dim:]
-    return torch.cat([qa.float(), qr], dim=-1).to(proj.dtype).contiguous()
+    return torch.cat([qa.float(), qr, torch.zeros(T, heads, pad)], dim=-1).to(proj.dtype).contiguous()
 
 
 def gla_recurrent(proj, q_col, k_col, v_col, z, bias, tau, qscale, state, seq_slot, seq_start, heads, dim, vdim, single=False):
@@ -206,7 +208,7 @@ def qk_norm_rope_append(qkv, num_heads, num_kv_heads, head_dim, q_gain, k_gain, 
 
 
 def attention(q, k_pool, v_pool, page_table, seq_slot, seq_start, seq_len, max_new, scale, window=0, sink=None, chunk=0,
-              softcap=0.0, dist_bias=None):
+              softcap=0.0, dist_bias=None, keep=0):
     T, H, Dh = q.shape
     KV, P = k_pool.shape[1], k_pool.shape[2]
     G = H // KV
@@ -218,6 +220,8 @@ def attention(q, k_pool, v_pool, page_table, seq_slot, seq_start, seq_len, max_n
             pos = n - (t1 - t0) + (t - t0)
             first = max(0, pos - window + 1) if window > 0 else (pos - pos % chunk if chunk > 0 else 0)
             idx = torch.arange(first, pos + 1)
+            if keep and window:
+                idx = torch.cat([torch.arange(0, min(keep, first)), idx])
             pages = page_table[slot, (idx // P).long()].long()
             assert (pages >= 0).all(), "read from an unmapped page"
             kk = k_pool[pages, :, (idx % P).long(), :].float()      # [n, KV, Dh]
@@ -347,8 +351,15 @@ def linear_gated(x, w_gate_up, block, kind="silu", limit=0.0, alpha=1.0):
     return gated_act(linear(x, w_gate_up), kind, block, limit, alpha)
 
 
-def moe_route(x, router, correction, top, score="softmax", groups=1, keep=1, group_top=2, scale=1.0, renormalize=True):
+def moe_route(x, router, correction, top, score="softmax", groups=1, keep=1, group_top=2, scale=1.0, renormalize=True,
+              bias=None):
     z = x.float() @ router.t()
+    if bias is not None:
+        z = z + bias
+    if score == "logits":
+        assert correction is None and groups == 1
+        best = torch.sort(z, dim=-1, descending=True, stable=True)
+        return best.indices[:, :top].to(torch.int32).contiguous(), torch.softmax(best.values[:, :top], dim=-1) * scale
     s = torch.softmax(z, dim=-1) if score == "softmax" else torch.sigmoid(z)
     c = s + correction
     if groups > 1:
@@ -486,7 +497,7 @@ def mlstm_head_norm_gate(o, gates, gain, eps, g, out_dtype):
 
 def qkv_prep(proj, q_col, k_col, v_col, heads, kv_heads, Dp, Dk, bias, rope_table, rot, pairs, unit, eps, k_pool, v_pool,
              page_table, tok_seq, tok_pos, seq_slot, write_kv=True, norm="", q_gain=None, k_gain=None, norm_eps=0.0,
-             q_factor=None, unit_v=False, Dv=0):
+             q_factor=None, unit_v=False, Dv=0, maps=1):
     T = proj.shape[0]
     x = proj.float()
     if bias is not None:
@@ -532,6 +543,9 @@ def qkv_prep(proj, q_col, k_col, v_col, heads, kv_heads, Dp, Dk, bias, rope_tabl
             k_pool[page, :, pos % P, :] = k[t].to(k_pool.dtype)
             if v is not None:
                 v_pool[page, :, pos % P, :] = v[t].to(v_pool.dtype)
+    if maps > 1:
+        own = (torch.arange(Dp) // (Dk // maps))[None, :] == torch.arange(maps)[:, None]
+        q = (q[:, :, None, :] * own).reshape(T, heads * maps, Dp)
     return q.to(proj.dtype).contiguous()
 
 
@@ -539,3 +553,24 @@ def softcap_(x, cap):
     if cap:
         x.copy_(cap * torch.tanh(x / cap))
     return x
+
+
+# ---- the parts of the seventh architecture --------------------------------------------------------------------------------
+def dyn_tanh(resid, alpha, gain, bias, out_dtype, delta=None, rows=None, then=None):
+    x = resid if rows is None else resid[rows.long()]
+    if delta is not None:
+        x = x + (delta if rows is None else delta[rows.long()]).float()
+        if rows is None:
+            resid.copy_(x)
+    return (torch.tanh(alpha * x) * gain + bias).to(out_dtype)
+
+
+def embed_dyn_tanh(ids, table, scale, alpha, gain, bias):
+    return torch.tanh(alpha * (table[ids.long()].float() * scale)) * gain + bias
+
+
+def pair_heads(x, lam, eps, gain, width, vdim):
+    f = x.float()
+    o = f[:, 0::2, :vdim] - lam * f[:, 1::2, :vdim]
+    o = o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps) * gain
+    return torch.nn.functional.pad(o, (0, width - vdim)).to(x.dtype).contiguous()
