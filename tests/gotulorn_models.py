@@ -182,18 +182,17 @@ def row_error(got, want):
     return float(np.sqrt((d * d).mean()) / max(np.sqrt((w * w).mean()), 1e-30))
 
 
-# (single rows, mean over all rows).  float32: rounding alone.  bfloat16: activations are rounded to 8 bits between the parts,
-# and where two of a router's outputs lie close together that rounding may choose another expert, and where a head's two maps
-# all but cancel its norm makes the rounding large: single rows are then further off, so the mean is held much tighter.
-BOUND = {"float32": (1e-4, 2e-5), "bfloat16": (6e-1, 5e-2)}
+# (nearly every row, mean over all rows, any row).  float32: rounding alone.  bfloat16: activations are rounded to 8 bits
+# between the parts, and where two of a router's outputs lie close together that rounding may choose another expert: such a
+# row is off by any amount, so one row in fifty may be, and the mean holds them all together.
+BOUND = {"float32": (1e-4, 2e-5, 1e-4), "bfloat16": (2.5e-1, 5e-2, 1.5)}
 
 
 def assert_rows_close(rows, want_by_request, dtype, what=""):
-    worst, total = 0.0, 0.0
-    for (rid, p), got in sorted(rows.items()):
-        err = row_error(got, want_by_request[rid][p])
-        worst, total = max(worst, err), total + err
-        assert err <= BOUND[dtype][0], f"{what}: request {rid} position {p}: error {err:.3e} exceeds {BOUND[dtype][0]:.1e}"
-    mean = total / max(len(rows), 1)
-    assert mean <= BOUND[dtype][1], f"{what}: mean error {mean:.3e} exceeds {BOUND[dtype][1]:.1e}"
-    return round(worst, 7), round(mean, 7)
+    most, mean_bound, any_row = BOUND[dtype]
+    errs = sorted(((row_error(got, want_by_request[rid][p]), rid, p) for (rid, p), got in rows.items()), reverse=True)
+    over = [e for e in errs if e[0] > most]
+    assert len(over) <= len(errs) // 50 and errs[0][0] <= any_row, f"{what}: {len(over)} of {len(errs)} rows over {most:.1e}: {over[:3]}"
+    mean = sum(e[0] for e in errs) / max(len(errs), 1)
+    assert mean <= mean_bound, f"{what}: mean error {mean:.3e} exceeds {mean_bound:.1e}"
+    return round(errs[0][0], 7), len(over), round(mean, 7)

@@ -136,16 +136,19 @@ def _plain_masked(q, k, v, scale, mask, positions):
                                                    (64, 20, 1, 31, 3), (48, 3, 1, 200, 129), (128, 2, 2, 129, 0), (64, 2, 1, 33, 300),
                                                    (22, 2, 1, 50, 32), (144, 6, 2, 40, 6), (128, 8, 2, 300, 1)])
 def test_attention_with_kept_first_tokens(D, Hq, KV, size, keep, dtype):
-    """Every other key is loud: its score stands out for every query that sees it, and its value is large, so that one key too
-    many or too few at either edge shows.  As a whole prompt, as portions that start inside a block of keys, and token by token
+    """A query that sees one of the loud keys hears nothing else: they stand further apart than the window is long, the first one
+    right behind the kept tokens, and the last kept token is loud where none of them is in sight, so that one key too many or
+    too few at either edge shows.  As a whole prompt, as portions that start inside a block of keys, and token by token
     around pages, blocks and the mask's edges, on every attention kernel; pages that nobody sees are not mapped."""
     from rust_inference_b200 import ops
     rng = np.random.default_rng(D + size)
     n, scale, mask = 420, 0.25, {"size": size, "keep_first": keep}
     k, v, q = (rng.standard_normal((n, h, D)) for h in (KV, KV, Hq))
+    q, k = q * 1.5 * D ** -0.25, k * 1.5 * D ** -0.25
     q[..., 0], k[..., 0] = 3.0, 0.0
-    k[rng.random(n) < 0.5, :, 0] = 5.0
-    v *= rng.uniform(0.5, 3.0, (n, 1, 1))
+    if keep:
+        k[keep - 1, :, 0] = 7.0
+    k[keep::size + 3, :, 0] = 13.0
     kt, vt, qt = _t(k, dtype), _t(v, dtype), _t(q, dtype)
     args = (_np(qt), _np(kt), _np(vt), scale)
     want = _plain_masked(*args, mask, range(n))
@@ -176,8 +179,11 @@ def test_attention_with_kept_first_tokens(D, Hq, KV, size, keep, dtype):
             got = ops.attention_prefill(one, kp, vp, table, slot, _i([0, 1]), length, 1, scale, size, keep=keep)
             _close(got, want[p:p + 1], dtype, f"prefill kernel, token {p}", **tol)
     _no_error()
-    for off in ({"size": size + 1, "keep_first": keep}, {"size": size, "keep_first": keep + 1}):
-        if keep + size < n:
+    masks = [{"size": size + 1, "keep_first": keep}, {"size": size, "keep_first": keep + 1}]
+    masks += [{"size": size - 1, "keep_first": keep}] if size > 1 else []
+    masks += [{"size": size, "keep_first": keep - 1}] if keep else []
+    for off in masks:
+        if keep + size + 8 < n:
             moved = _plain_masked(*args, off, range(n))
             assert np.abs(moved - want).max() > 0.1 * np.abs(want).max(), "an edge that is one token off would not show"
 
