@@ -18,16 +18,18 @@ steps end at exactly 4,096 tokens.  One JSON line is printed:
   points     decode tokens a second at batch 1 and 64 (device-timed), and the same through
              the Python entry point (e2e_b1, e2e_b64)
 
-    python bench.py --design ranudra|pitenex|kagatar|puratar|zavevik [--size small|large]
+    python bench.py --design ranudra|pitenex|kagatar|puratar|zavevik|gotulorn [--size small|large]
 
 measures another design (Ranudra: latent attention, gated linear attention, hyper-connections; Pitenex: chunked attention
 with a sink beside the gated delta rule, dense and routed feed-forwards; Kagatar: three kinds of attention with biases
 beside a clamped-swish feed-forward behind two gains over one RMS statistic; Puratar: norms in front of and behind every
 sublayer, attention with a gate per head or beside the matrix memory of xLSTM, dense and routed feed-forwards; Zavevik:
 norms behind the sublayers only, attention with a distance bias, borrowed keys and values, the delta rule with one decay
-per head, experts by token id, a token-fed sublayer) at layer
+per head, experts by token id, a token-fed sublayer; Gotulorn: Dynamic Tanh norms, differential attention with a window
+beside kept first tokens, latent attention, dense and routed feed-forwards) at layer
 sizes that resemble a real model's, beside a Qwen3 model of the same width and depth (Puratar and Zavevik: beside the
-Pitenex model of the same width and depth, the closest design): decode at batch 8 and a
+Pitenex model of the same width and depth, the closest design; Gotulorn: beside the Pitenex model, which has the like
+feed-forwards and attention, and the Ranudra model, which has the like latent attention): decode at batch 8 and a
 prompt step of 2,048 tokens, device-timed, and the device time of every section of both steps from eager runs with
 the section timers on, with the bytes or flops of the sections that have a roofline.  One JSON line.
 
@@ -373,10 +375,30 @@ def zavevik_config(z) -> dict:
             "layers": layers}
 
 
+def gotulorn_config(z) -> dict:
+    """Layers in turns of three: differential attention (half as many heads as the width has parts of 128, each with two maps
+    of 64 and a value of 128, four heads per key/value head, a window of 2,048 beside 4 kept tokens), latent attention (per
+    head 128 plain and 64 rotated elements, a latent of 192), differential attention over the keys and values of the first.
+    Feed-forwards take turns: dense, and routed (16 experts of an eighth of the dense width, 4 per token)."""
+    D, H = z["width"], z["heads"]
+    inter = -(-(2 * z["ff"] // 3) // 256) * 256          # three matrices of a gated feed-forward against two
+    ffs = [{"kind": "dense", "ff": inter, "limit": 7.0},
+           {"kind": "moe", "router": {"experts": 16, "top": 4}, "expert": {"ff": inter // 8}}]
+    pairs = {"heads": H, "kv_heads": max(1, H // 4), "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "diff": 0.5,
+             "mask": {"size": 2048, "keep_first": 4}}
+    lat = {"heads": H, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 192, "scale": 192 ** -0.5,
+           "rot": {"base": 500000.0, "dims": 64}}
+    layers = []
+    for i in range(0, z["layers"] // 3 * 3, 3):
+        layers += [{"type": "attention", "mixer": pairs, "mlp": ffs[i % 2]}, {"type": "latent_attention", "mixer": lat, "mlp": ffs[(i + 1) % 2]},
+                   {"type": "attention", "mixer": dict(pairs, kv_from=i), "mlp": ffs[i % 2]}]
+    return {"architecture": "Gotulorn", "vocab": z["vocab"], "width": D, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6}, "layers": layers}
+
+
 DESIGNS = {"ranudra": ranudra_config, "pitenex": pitenex_config, "kagatar": kagatar_config, "puratar": puratar_config,
-           "zavevik": zavevik_config}
-# the model that a design is measured beside, where it is not the Qwen3 model of equal size: the closest design
-BESIDE = {"puratar": "pitenex", "zavevik": "pitenex"}
+           "zavevik": zavevik_config, "gotulorn": gotulorn_config}
+# the models that a design is measured beside, where it is not the Qwen3 model of equal size: the closest designs
+BESIDE = {"puratar": ("pitenex",), "zavevik": ("pitenex",), "gotulorn": ("pitenex", "ranudra")}
 
 
 def qwen3_like(z) -> dict:
@@ -403,8 +425,9 @@ def run_design(a) -> int:
     clocks.start()
     windows = []
     out = {}
-    other = BESIDE.get(a.design, "qwen3")
-    for label, cfg in ((a.design, DESIGNS[a.design](z)), (other, DESIGNS[other](z) if other in DESIGNS else qwen3_like(z))):
+    others = BESIDE.get(a.design, ("qwen3",))
+    for label in (a.design,) + others:
+        cfg = DESIGNS[label](z) if label in DESIGNS else qwen3_like(z)
         t_model = time.time()
         model = Model.from_random(cfg, seed=1, dtype="bfloat16", device=dev)
         V = model.spec.vocab_size
@@ -490,9 +513,9 @@ def run_design(a) -> int:
         "ms_per_step": r["decode_ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
         "dtype": "bf16", "data": "synthetic: random-init weights, uniform random token ids", "design": a.design,
         "config": dict(z, size=a.size, global_batch=B, seq_len=ctx, prefill_tokens=T, parallelism="1 GPU", peaks=peak_src,
-                       beside=f"a {other.capitalize()} model of the same width and depth (weight_bytes of both are given)"),
+                       beside=" and ".join(f"a {o.capitalize()} model" for o in others) + " of the same width and depth (weight_bytes of all are given)"),
         "peaks": {"hbm_gbs": hbm_gbs, "bf16_tflops": bf16_tflops},
-        a.design: r, other: out[other], "clocks": clocks.summary(windows), "gpu_launches": r["decode_launches"] * K,
+        **out, "clocks": clocks.summary(windows), "gpu_launches": r["decode_launches"] * K,
         "impl": "ours",
     }
     print(json.dumps(line))
