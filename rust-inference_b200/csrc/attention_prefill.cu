@@ -68,10 +68,10 @@ __device__ __forceinline__ void load_kv_block(PrefillSmem& sm, int buf, int kb, 
 
 __global__ void __launch_bounds__(32 * PF_WARPS)
 attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool, const bf16* __restrict__ v_pool,
-                         bf16* __restrict__ out, const int* __restrict__ page_table, const int* __restrict__ seq_slot,
+                         void* __restrict__ out, const int* __restrict__ page_table, const int* __restrict__ seq_slot,
                          const int* __restrict__ seq_start, const int* __restrict__ seq_len, int H, int KV, int mpps,
                          int num_pages, float scale_log2, int window, const float* __restrict__ sink, int shared_kv,
-                         int v_dims, int* __restrict__ err, float cap_raw, DistBias bias, int keep) {
+                         int v_dims, int* __restrict__ err, float cap_raw, DistBias bias, int keep, int out_f32) {
     // keep: beside a window, the sequence's first keys that every query sees
     // bias: a distance bias per head, added after the cap (in units of log2 here, like the scaled scores)
     // cap_raw > 0: a soft cap on the scores in unscaled units (cap / scale), applied before the scale and the mask.
@@ -222,7 +222,14 @@ attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_
         int row = warp * 16 + quad + r * 8;
         if (row >= rows) continue;
         float inv = 1.0f / l[r];
-        bf16* dst = out + ((size_t)(t_begin + r_base + row) * H + h) * PF_DH;
+        const size_t at = ((size_t)(t_begin + r_base + row) * H + h) * PF_DH;
+        if (out_f32) {
+            float* dst = (float*)out + at;
+#pragma unroll
+            for (int t = 0; t < PF_DH / 8; t++) *(float2*)(dst + t * 8 + qc * 2) = make_float2(o[t][r * 2] * inv, o[t][r * 2 + 1] * inv);
+            continue;
+        }
+        bf16* dst = (bf16*)out + at;
 #pragma unroll
         for (int t = 0; t < PF_DH / 8; t++) {
             __nv_bfloat162 v = __floats2bfloat162_rn(o[t][r * 2] * inv, o[t][r * 2 + 1] * inv);
@@ -241,8 +248,9 @@ extern "C" int ri_attention_prefill(const void* q, const void* k_pool, const voi
                                     const int* page_table, const int* seq_slot, const int* seq_start,
                                     const int* seq_len, int seqs, int max_new, int H, int KV, int Dh, int mpps,
                                     int page_size, int num_pages, float scale, int window, const float* sink,
-                                    int v_dims, float softcap, const float* dist_bias, int bias_len, int keep, int* err_flag,
+                                    int v_dims, float softcap, const float* dist_bias, int bias_len, int keep, int out_f32, int* err_flag,
                                     cudaStream_t stream) {
+    // out_f32: out is float32 (for a kernel behind this one that puts results together before it rounds)
     if (seqs == 0 || max_new == 0) return 0;
     RI_REQUIRE(keep >= 0, "attention_prefill: %d kept keys", keep);
     if (window <= 0) keep = 0;                 // nothing is out of sight, or the mask is one of chunks
@@ -267,9 +275,9 @@ extern "C" int ri_attention_prefill(const void* q, const void* k_pool, const voi
     }
     dim3 grid((max_new + PF_BM - 1) / PF_BM, H, seqs);
     attention_prefill_kernel<<<grid, 32 * PF_WARPS, smem, stream>>>(
-        (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, (bf16*)out, page_table, seq_slot, seq_start, seq_len,
+        (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, out, page_table, seq_slot, seq_start, seq_len,
         H, KV, mpps, num_pages, scale * 1.4426950408889634f, window, sink, shared_kv, v_dims, err_flag,
-        softcap > 0.0f ? softcap / scale : 0.0f, DistBias{dist_bias, bias_len}, keep);
+        softcap > 0.0f ? softcap / scale : 0.0f, DistBias{dist_bias, bias_len}, keep, out_f32);
     RI_CHECK_LAUNCH("attention_prefill");
     return 0;
 }

@@ -53,12 +53,20 @@
 // it sees keys max(0, pos-window+1)..pos and, beside a window, the sequence's first `keep` keys.  A query's result depends on its position
 // and its place in the step, not on the batch.
 //
+// Differential attention (PAIR, a variant of its own; pair_heads.cuh has the formula): an item is ONE query tile of 128 tokens
+// and one pair of heads, the two maps over the same values; tile 0 is the first map, tile 1 the second.  Both see the same
+// blocks of keys.  A map's query is zero outside its own half of the row, so its product with the keys takes only the k steps
+// of that half.  At the end of an item tile 1's threads hand the reciprocals of their rows' sums over in shared memory, and tile
+// 0's threads read both outputs from tensor memory (a thread reaches its row's lane in the columns of either tile), take the
+// difference, norm it and store it: nothing is rounded before that.
+//
 // Compile with -DRI_HEAD_DIM=64 or 128.  Page size is 32.
 // Formula: thanhauco/rust-inference src/attention.rs:4-8, 111-150.
 #include "common.cuh"
 #include "mma_helpers.cuh"
 #include "softcap.cuh"
 #include "distance_bias.cuh"
+#include "pair_heads.cuh"
 #include <cuda.h>
 #include <float.h>
 
@@ -270,8 +278,9 @@ struct TcTail {
     unsigned long long q_full[2], q_empty[2], o_free[2];
     unsigned tmem_base;
     volatile int dead;
+    float pair_inv[TC_BM];              // 1 / (sum of the row's weights) of tile 1, for tile 0's threads
 };
-#define TC_SMEM_BYTES (TC_OFF_TAIL + 448)
+#define TC_SMEM_BYTES (TC_OFF_TAIL + 448 + TC_BM * 4)
 #define TC_TMEM_COLS 512
 #define TC_S_COL(t, b) (((t) * 2 + (b)) * TC_BN)       // two S buffers per tile
 #define TC_O_COL(t) (4 * TC_BN + (t) * 128)
@@ -297,33 +306,37 @@ struct TcWork {
     float cap_raw;              // a soft cap on the scores in unscaled units (cap / scale), 0 for none
     DistBias bias;              // a distance bias per head on the scores (table null: none)
     float inv_scale;            // 1 / scale: the bias in unscaled units
+    PairOut pair;               // heads 2 h and 2 h + 1 are two maps of one head
+    int pair_dim;               // elements of one map's query and key (map m's are m pair_dim .. of the row)
 };
 // The items in the order (group of rows: late ones, which see the most keys, first; sequence; head).  Block c of G
 // takes item k G + c in its round k when k is even and item k G + G - 1 - c when k is odd, so the block that drew
 // the heaviest item of one round draws the lightest of the next.  False: no item for this block in this round.
+template <bool PAIR>
 __device__ __forceinline__ bool tc_item(const TcWork& w, int k, TcItem& it) {
     const int G = (int)gridDim.x;
     const int id = (k & 1) ? k * G + G - 1 - (int)blockIdx.x : k * G + (int)blockIdx.x;
     if (id >= w.n_items) return false;
-    const int per = w.seqs * w.H;
+    const int heads = PAIR ? w.H / 2 : w.H;
+    const int per = w.seqs * heads;
     const int g_rev = id / per, rem = id - g_rev * per;
-    const int b = rem / w.H;
-    it.h = rem - b * w.H;
+    const int b = rem / heads;
+    it.h = (rem - b * heads) * (PAIR ? 2 : 1);
     const int group = w.groups_max - 1 - g_rev;
-    constexpr int ROWS = TC_TILES * TC_BM;
+    constexpr int ROWS = PAIR ? TC_BM : TC_TILES * TC_BM;
     const int t_begin = w.seq_start[b], n_new = w.seq_start[b + 1] - t_begin;
     if (group * ROWS >= n_new) return false;
     it.len = w.seq_len[b];
     const int r_base = group * ROWS;
     it.t_first = t_begin + r_base;
     it.rows = min(ROWS, n_new - r_base);
-    it.n_tiles = it.rows > TC_BM ? 2 : 1;
+    it.n_tiles = PAIR || it.rows > TC_BM ? 2 : 1;
     it.pos_first = it.len - n_new + r_base;
     it.pos_last = it.pos_first + it.rows - 1;
     it.key_lo = ri_first_visible(it.pos_first, w.window);
     it.runs = RiRuns::of(it.key_lo / TC_BN, w.keep, TC_BN);
     it.n_blocks = it.pos_last / TC_BN + 1 - it.runs.shift;
-    it.n_blocks_0 = it.n_tiles > 1 ? min(it.n_blocks, (it.pos_first + TC_BM - 1) / TC_BN + 1 - it.runs.shift) : it.n_blocks;
+    it.n_blocks_0 = !PAIR && it.n_tiles > 1 ? min(it.n_blocks, (it.pos_first + TC_BM - 1) / TC_BN + 1 - it.runs.shift) : it.n_blocks;
     it.kvh = it.h / (w.H / w.KV);
     it.table = w.page_table + (size_t)w.seq_slot[b] * w.mpps;
     return true;
@@ -334,8 +347,8 @@ __device__ __forceinline__ int tc_tile_blocks(const TcItem& it, int t) {
     return t < it.n_tiles ? (t == 0 ? it.n_blocks_0 : it.n_blocks) : 0;
 }
 
-// BIAS: with a distance bias (a variant of its own, so that the others keep their registers)
-template <bool BIAS>
+// BIAS: with a distance bias (a variant of its own, so that the others keep their registers); PAIR: see the top
+template <bool BIAS, bool PAIR>
 __global__ void __launch_bounds__(TC_THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                              const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out, const TcWork work,
@@ -409,7 +422,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             int kv_base = 0, n_it = 0;            // blocks of keys and items before the one at hand
             for (int k = 0; k < rounds && !dead; k++) {
                 TcItem it;
-                if (!tc_item(work, k, it)) continue;
+                if (!tc_item<PAIR>(work, k, it)) continue;
                 // both query tiles, once the products of the item before have read theirs (rows past the sequence's
                 // belong to the next one or read as zeros past the last token: they are computed and never stored)
                 auto load_q = [&]() {
@@ -420,8 +433,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                         tc_expect_tx(&tail.q_full[t], TC_Q_TILE_BYTES);
 #pragma unroll
                         for (int sl = 0; sl < TC_SLABS; sl++)
-                            tc_tma_2d(smem + TC_OFF_Q + t * TC_Q_TILE_BYTES + sl * TC_Q_SLAB, &map_q, it.h * TC_DH + sl * 64,
-                                      it.t_first + t * TC_BM, &tail.q_full[t]);
+                            tc_tma_2d(smem + TC_OFF_Q + t * TC_Q_TILE_BYTES + sl * TC_Q_SLAB, &map_q,
+                                      (it.h + (PAIR ? t : 0)) * TC_DH + sl * 64, it.t_first + (PAIR ? 0 : t * TC_BM), &tail.q_full[t]);
                         q_started = n_it * TC_TILES + t + 1;
                     }
                 };
@@ -474,6 +487,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 vd[i] = v_base + (unsigned)((i * 16 * 128) >> 4);
             }
             const unsigned o_col = tmem + TC_O_COL(t);
+            // the k steps in which this tile's queries are not zero
+            const int k_from = PAIR ? t * work.pair_dim / 16 : 0, k_to = PAIR ? ((t + 1) * work.pair_dim + 15) / 16 : TC_DH / 16;
             bool dead = false;
             auto wait = [&](unsigned long long* bar, unsigned parity) {
                 if (!dead && !tc_mbar_wait(bar, parity)) { atomicExch(err, 5); tail.dead = 1; dead = true; }
@@ -484,7 +499,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             int c = 0, kv_base = 0, n_it = 0, n_mine = 0;
             for (int k = 0; k < rounds && !dead; k++) {
                 TcItem it;
-                if (!tc_item(work, k, it)) continue;
+                if (!tc_item<PAIR>(work, k, it)) continue;
                 const int my_blocks = tc_tile_blocks(it, t);
                 wait(&tail.q_full[t], (unsigned)(n_it & 1));
                 // S_t of the item's block jb = Q_t K^T into S buffer (c + jb) & 1, once the threads hold what that buffer
@@ -497,7 +512,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     const unsigned long long off = (unsigned long long)(st * (TC_KV_BYTES >> 4));
                     const unsigned s_col = tmem + TC_S_COL(t, idx & 1);
 #pragma unroll
-                    for (int i = 0; i < TC_DH / 16; i++) umma_bf16(s_col, qd[i], kd[i] + off, IDESC_QK, i > 0);
+                    for (int i = 0; i < TC_DH / 16; i++) {
+                        if (PAIR && (i < k_from || i >= k_to)) continue;
+                        umma_bf16(s_col, qd[i], kd[i] + off, IDESC_QK, PAIR ? i > k_from : i > 0);
+                    }
                     umma_commit(&tail.s_full[t][idx & 1]);
                     umma_commit(&tail.k_empty[st]);                          // this tile is done with the keys of block jb
                     if (jb + 1 == my_blocks) umma_commit(&tail.q_empty[t]);  // ... and with the item's queries
@@ -550,16 +568,17 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         int c = 0, kv_base = 0;
         for (int k = 0; k < rounds; k++) {
             TcItem it;
-            if (!tc_item(work, k, it)) continue;
+            if (!tc_item<PAIR>(work, k, it)) continue;
             const int my_blocks = tc_tile_blocks(it, t);
             if (my_blocks == 0) {
                 kv_base += it.n_blocks;
                 continue;
             }
             const int len = it.len, key_lo = it.key_lo, pos_first = it.pos_first, pos_last = it.pos_last;
-            const int my_pos = pos_first + t * TC_BM + row;
-            const int tile_first = pos_first + t * TC_BM, tile_last = min(tile_first + TC_BM - 1, pos_last);
-            const bool real_row = t * TC_BM + row < it.rows;
+            const int row_of = PAIR ? row : t * TC_BM + row;           // the row within the item
+            const int my_pos = pos_first + row_of;
+            const int tile_first = my_pos - row, tile_last = min(tile_first + TC_BM - 1, pos_last);
+            const bool real_row = row_of < it.rows;
             float m = -FLT_MAX, l = 0.0f;
             for (int j = 0; j < my_blocks; j++) {
                 const int kb = it.runs.block(j), idx = c + j, gj = kv_base + j;
@@ -734,6 +753,60 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             // (m is the running maximum in units of log2, possibly a little below the true one: l and O are both relative to it)
             if (work.sink && m != -FLT_MAX) l += ex2_approx(work.sink[it.h] * 1.4426950408889634f - m);
             const float inv = 1.0f / l;
+            if (PAIR) {
+                // both tiles' threads have the item's outputs in tensor memory behind this barrier
+                if (t == 1) tail.pair_inv[row] = inv;
+                tc_fence_before();
+                asm volatile("bar.sync 1, %0;\n" ::"n"(32 * 4 * TC_TILES) : "memory");
+                tc_fence_after();
+                if (t == 0) {
+                    const PairOut& pr = work.pair;
+                    const float inv1 = pr.lam * tail.pair_inv[row];
+                    float ss = 0.0f;
+#pragma unroll
+                    for (int cc = 0; cc < TC_DH / 32; cc++) {
+                        float a[32], b[32];
+                        tmem_ld32(tmem_row + TC_O_COL(0) + cc * 32, a);
+                        tmem_ld32(tmem_row + TC_O_COL(1) + cc * 32, b);
+#pragma unroll
+                        for (int i = 0; i < 32; i++) {
+                            const float o = a[i] * inv - b[i] * inv1;
+                            ss += cc * 32 + i < pr.vdim ? o * o : 0.0f;
+                        }
+                    }
+                    const float f = pr.gain / sqrtf(ss / (float)pr.vdim + pr.eps);
+                    bf16* dst = out + ((size_t)(it.t_first + (mine ? row : 0)) * (H / 2) + it.h / 2) * pr.width;
+#pragma unroll
+                    for (int cc = 0; cc < TC_DH / 32; cc++) {
+                        float a[32], b[32];
+                        tmem_ld32(tmem_row + TC_O_COL(0) + cc * 32, a);
+                        tmem_ld32(tmem_row + TC_O_COL(1) + cc * 32, b);
+                        if (mine) {
+#pragma unroll
+                            for (int i = 0; i < 32; i += 8) {
+                                if (cc * 32 + i >= pr.width) continue;
+                                float y[8];
+#pragma unroll
+                                for (int e = 0; e < 8; e++)
+                                    y[e] = cc * 32 + i + e < pr.vdim ? (a[i + e] * inv - b[i + e] * inv1) * f : 0.0f;
+                                *(uint4*)(dst + cc * 32 + i) = make_uint4(pack_bf16(y[0], y[1]), pack_bf16(y[2], y[3]),
+                                                                          pack_bf16(y[4], y[5]), pack_bf16(y[6], y[7]));
+                            }
+                        }
+                    }
+                    // both outputs have been read: the next item's first products may overwrite them (tile 1's threads write
+                    // pair_inv again only behind the next item's products)
+                    tc_fence_before();
+                    __syncwarp();
+                    if (lane == 0) {
+                        asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(smem_u32(&tail.o_free[0])) : "memory");
+                        asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(smem_u32(&tail.o_free[1])) : "memory");
+                    }
+                }
+                c += my_blocks;
+                kv_base += it.n_blocks;
+                continue;
+            }
             bf16* dst = out + ((size_t)(it.t_first + (mine ? t * TC_BM + row : 0)) * H + it.h) * TC_DH;
 #pragma unroll
             for (int cc = 0; cc < TC_DH / 32; cc++) {
@@ -831,8 +904,11 @@ extern "C" int ri_attention_prefill_tc(const void* q, const void* k_pool, const 
                                        const int* page_table, const int* seq_slot, const int* seq_start,
                                        const int* seq_len, int tokens, int seqs, int max_new, int H, int KV, int Dh, int mpps,
                                        int page_size, int num_pages, float scale, int window, const float* sink,
-                                       float softcap, const float* dist_bias, int bias_len, int keep, int* err_flag,
-                                       cudaStream_t stream) {
+                                       float softcap, const float* dist_bias, int bias_len, int keep, int pair_width,
+                                       int pair_vdim, int pair_dim, float pair_lam, float pair_eps, float pair_gain,
+                                       int* err_flag, cudaStream_t stream) {
+    // pair_width > 0: heads 2 h and 2 h + 1 are the two maps of differential attention, queries and keys of map m at elements
+    // m pair_dim .. (m + 1) pair_dim - 1 of a row (zeros elsewhere in a query); out [tokens, H / 2, pair_width]
     // keep: beside a window, the sequence's first keys that every query sees
     // dist_bias (float32, bias_len entries a head between their padding) or null: added to the score by the query's distance to the key (distance_bias.cuh)
     // softcap > 0: score <- softcap * tanh(score / softcap) after the scale (0: none)
@@ -848,8 +924,14 @@ extern "C" int ri_attention_prefill_tc(const void* q, const void* k_pool, const 
     RI_REQUIRE(scale > 0.0f, "attention_prefill_tc: the score scale must be positive");
     RI_REQUIRE((((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)out) & 15) == 0,
                "attention_prefill_tc: q, out and the pools must be 16-byte aligned");
-    const int groups_max = (max_new + TC_TILES * TC_BM - 1) / (TC_TILES * TC_BM);
-    const long long n_items = (long long)groups_max * seqs * H;
+    const bool paired = pair_width > 0;
+    RI_REQUIRE(!paired || (H % 2 == 0 && (H / KV) % 2 == 0 && pair_width % 8 == 0 && pair_width <= TC_DH && pair_vdim > 0 &&
+                           pair_vdim <= pair_width && pair_dim > 0 && 2 * pair_dim <= TC_DH && !sink && !dist_bias),
+               "attention_prefill_tc: pairs of %d heads over %d kv heads, maps of %d, %d elements in rows of %d", H, KV, pair_dim,
+               pair_vdim, pair_width);
+    const int rows_item = paired ? TC_BM : TC_TILES * TC_BM;
+    const int groups_max = (max_new + rows_item - 1) / rows_item;
+    const long long n_items = (long long)groups_max * seqs * (paired ? H / 2 : H);
     RI_REQUIRE(n_items < (1ll << 30), "attention_prefill_tc: %lld work items", n_items);
     RI_REQUIRE((long long)num_pages * KV * TC_PAGE < (1ll << 31), "attention_prefill_tc: a pool of %d pages", num_pages);
     CUtensorMap map_q, map_k, map_v;
@@ -862,8 +944,9 @@ extern "C" int ri_attention_prefill_tc(const void* q, const void* k_pool, const 
     static bool configured = false;
     static int sms = 0;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC_SMEM_BYTES);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_prefill_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC_SMEM_BYTES);
+        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC_SMEM_BYTES);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_prefill_tc_kernel<true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC_SMEM_BYTES);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_prefill_tc_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC_SMEM_BYTES);
         if (e != cudaSuccess) RI_FAIL((int)e, "attention_prefill_tc: %s", cudaGetErrorString(e));
         int dev = 0;
         cudaGetDevice(&dev);
@@ -888,15 +971,16 @@ extern "C" int ri_attention_prefill_tc(const void* q, const void* k_pool, const 
     work.cap_raw = softcap > 0.0f ? softcap / scale : 0.0f;
     work.bias = DistBias{dist_bias, bias_len};
     work.inv_scale = 1.0f / scale;
+    work.pair = PairOut{paired ? 1 : 0, pair_lam, pair_eps, pair_gain, pair_vdim, pair_width};
+    work.pair_dim = pair_dim;
     // one block per SM (the kernel's shared memory allows no second), each taking its items one after the other
     const int blocks = n_items < sms ? (int)n_items : sms;
     const float scale_log2 = scale * 1.4426950408889634f;
-    if (dist_bias)
-        attention_prefill_tc_kernel<true><<<blocks, TC_THREADS, TC_SMEM_BYTES, stream>>>(map_q, map_k, map_v, (bf16*)out, work,
-                                                                                         num_pages, scale_log2, err_flag);
-    else
-        attention_prefill_tc_kernel<false><<<blocks, TC_THREADS, TC_SMEM_BYTES, stream>>>(map_q, map_k, map_v, (bf16*)out, work,
-                                                                                          num_pages, scale_log2, err_flag);
+#define TC_GO(B, P) attention_prefill_tc_kernel<B, P><<<blocks, TC_THREADS, TC_SMEM_BYTES, stream>>>(map_q, map_k, map_v, (bf16*)out, work, num_pages, scale_log2, err_flag)
+    if (paired) TC_GO(false, true);
+    else if (dist_bias) TC_GO(true, false);
+    else TC_GO(false, false);
+#undef TC_GO
     RI_CHECK_LAUNCH("attention_prefill_tc");
     return 0;
 }

@@ -49,7 +49,7 @@ SOURCES: Dict[str, Tuple[str, ...]] = {
     "attention_prefill": ("attention_prefill.cu", "common.cuh", "mma_helpers.cuh", "softcap.cuh", "distance_bias.cuh"),
     "linear_skinny": ("linear_skinny.cu", "common.cuh", "mma_helpers.cuh", "linear_skinny_geometry.cuh"),
     "linear_stream_tc": ("linear_stream_tc.cu", "common.cuh", "mma_helpers.cuh"),
-    "attention_prefill_tc": ("attention_prefill_tc.cu", "common.cuh", "mma_helpers.cuh", "softcap.cuh", "distance_bias.cuh"),
+    "attention_prefill_tc": ("attention_prefill_tc.cu", "common.cuh", "mma_helpers.cuh", "softcap.cuh", "distance_bias.cuh", "pair_heads.cuh"),
     "attention_decode_noalloc": ("attention_decode_noalloc.cu", "attention_decode_noalloc.h", "attention_decode.cu",
                                  "common.cuh", "mma_helpers.cuh", "softcap.cuh", "distance_bias.cuh", "pair_heads.cuh"),
     "random_fill": ("random_fill.cu", "common.cuh", "random_fill.cuh"),

@@ -7,9 +7,9 @@
 #define PH_WARPS 8
 #define PH_PER_LANE 16           // elements a lane keeps in registers: heads of up to 512
 
-template <typename T, int N>
+template <typename T, typename TO, int N>
 __global__ void __launch_bounds__(32 * PH_WARPS)
-pair_heads_kernel(const T* __restrict__ x, T* __restrict__ y, PairOut p, long long heads, int Dp) {
+pair_heads_kernel(const T* __restrict__ x, TO* __restrict__ y, PairOut p, long long heads, int Dp) {
     pdl_trigger();
     pdl_wait();
     const int lane = threadIdx.x & 31;
@@ -26,7 +26,7 @@ pair_heads_kernel(const T* __restrict__ x, T* __restrict__ y, PairOut p, long lo
         ss += o[i] * o[i];
     }
     const float f = p.gain / sqrtf(warp_sum(ss) / (float)p.vdim + p.eps);
-    T* dst = y + (size_t)h * p.width;
+    TO* dst = y + (size_t)h * p.width;
 #pragma unroll
     for (int i = 0; i < N; i++) {
         const int d = i * 32 + lane;
@@ -34,10 +34,11 @@ pair_heads_kernel(const T* __restrict__ x, T* __restrict__ y, PairOut p, long lo
     }
 }
 
-// bfloat16 rows of whole 16-byte pieces: GROUP lanes (a power of two) per head, eight neighbouring elements per lane
+// rows of whole 16-byte pieces, float32 in and bfloat16 out: GROUP lanes (a power of two) per head, eight neighbouring
+// elements per lane
 template <int GROUP>
 __global__ void __launch_bounds__(32 * PH_WARPS)
-pair_heads8_kernel(const __nv_bfloat16* __restrict__ x, __nv_bfloat16* __restrict__ y, PairOut p, long long heads, int Dp) {
+pair_heads8_kernel(const float* __restrict__ x, __nv_bfloat16* __restrict__ y, PairOut p, long long heads, int Dp) {
     pdl_trigger();
     pdl_wait();
     const int ln = threadIdx.x % GROUP, d = 8 * ln;
@@ -47,16 +48,12 @@ pair_heads8_kernel(const __nv_bfloat16* __restrict__ x, __nv_bfloat16* __restric
 #pragma unroll
     for (int j = 0; j < 8; j++) o[j] = 0.0f;
     if (live && d < Dp) {
-        const uint4 ra = *reinterpret_cast<const uint4*>(x + (size_t)h * 2 * Dp + d);
-        const uint4 rb = *reinterpret_cast<const uint4*>(x + (size_t)h * 2 * Dp + Dp + d);
-        const __nv_bfloat162* a2 = reinterpret_cast<const __nv_bfloat162*>(&ra);
-        const __nv_bfloat162* b2 = reinterpret_cast<const __nv_bfloat162*>(&rb);
+        const float4* pa = reinterpret_cast<const float4*>(x + (size_t)h * 2 * Dp + d);
+        const float4* pb = reinterpret_cast<const float4*>(x + (size_t)h * 2 * Dp + Dp + d);
+        const float4 a0 = pa[0], a1 = pa[1], b0 = pb[0], b1 = pb[1];
+        const float fa[8] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w}, fb[8] = {b0.x, b0.y, b0.z, b0.w, b1.x, b1.y, b1.z, b1.w};
 #pragma unroll
-        for (int j = 0; j < 4; j++) {
-            const float2 fa = __bfloat1622float2(a2[j]), fb = __bfloat1622float2(b2[j]);
-            o[2 * j] = d + 2 * j < p.vdim ? fa.x - p.lam * fb.x : 0.0f;
-            o[2 * j + 1] = d + 2 * j + 1 < p.vdim ? fa.y - p.lam * fb.y : 0.0f;
-        }
+        for (int j = 0; j < 8; j++) o[j] = d + j < p.vdim ? fa[j] - p.lam * fb[j] : 0.0f;
     }
     float ss = 0.0f;
 #pragma unroll
@@ -77,20 +74,21 @@ pair_heads8_kernel(const __nv_bfloat16* __restrict__ x, __nv_bfloat16* __restric
 }
 
 extern "C" int ri_pair_heads(const void* x, void* y, float lam, float eps, float gain, int tokens, int H, int Dp, int width,
-                             int vdim, int dtype, cudaStream_t stream) {
+                             int vdim, int dtype, int out_dtype, cudaStream_t stream) {
+    // dtype: of x; out_dtype: of y (the same, or bfloat16 behind float32)
     if (tokens == 0) return 0;
     RI_REQUIRE(tokens > 0 && H > 0 && vdim > 0 && vdim <= Dp && vdim <= width, "pair_heads: bad sizes");
     RI_REQUIRE(width <= 32 * PH_PER_LANE, "pair_heads: rows of %d elements exceed the limit %d", width, 32 * PH_PER_LANE);
     const PairOut p{1, lam, eps, gain, vdim, width};
     const long long heads = (long long)tokens * H;
-    if (dtype == RI_DTYPE_BF16 && Dp % 8 == 0 && width % 8 == 0 && width <= Dp && Dp <= 256 && (((uintptr_t)x | (uintptr_t)y) & 15) == 0) {
+    if (dtype == RI_DTYPE_F32 && out_dtype == RI_DTYPE_BF16 && Dp % 8 == 0 && width % 8 == 0 && width <= Dp && Dp <= 256 && (((uintptr_t)x | (uintptr_t)y) & 15) == 0) {
         int group = 1;
         while (group < Dp / 8) group <<= 1;
         const int per = 32 * PH_WARPS / group;
         const dim3 grid((unsigned)((heads + per - 1) / per));
 #define PH8(G)                                                                                                            \
     if (group == G)                                                                                                       \
-        ri_launch_pdl(pair_heads8_kernel<G>, grid, dim3(32 * PH_WARPS), 0, stream, (const __nv_bfloat16*)x, (__nv_bfloat16*)y, \
+        ri_launch_pdl(pair_heads8_kernel<G>, grid, dim3(32 * PH_WARPS), 0, stream, (const float*)x, (__nv_bfloat16*)y, \
                       p, heads, Dp)
         PH8(1);
         PH8(2);
@@ -103,12 +101,17 @@ extern "C" int ri_pair_heads(const void* x, void* y, float lam, float eps, float
         return 0;
     }
     const dim3 grid((unsigned)((heads + PH_WARPS - 1) / PH_WARPS));
-#define PH_GO(T, N) ri_launch_pdl(pair_heads_kernel<T, N>, grid, dim3(32 * PH_WARPS), 0, stream, (const T*)x, (T*)y, p, heads, Dp)
-    if (dtype == RI_DTYPE_F32) {
-        if (width <= 128) PH_GO(float, 4); else PH_GO(float, PH_PER_LANE);
-    } else if (dtype == RI_DTYPE_BF16) {
-        if (width <= 128) PH_GO(__nv_bfloat16, 4); else PH_GO(__nv_bfloat16, PH_PER_LANE);
-    } else RI_FAIL(-1, "pair_heads: unknown dtype %d", dtype);
+#define PH_GO(T, TO)                                                                                                         \
+    do {                                                                                                                     \
+        if (width <= 128)                                                                                                    \
+            ri_launch_pdl(pair_heads_kernel<T, TO, 4>, grid, dim3(32 * PH_WARPS), 0, stream, (const T*)x, (TO*)y, p, heads, Dp); \
+        else                                                                                                                 \
+            ri_launch_pdl(pair_heads_kernel<T, TO, PH_PER_LANE>, grid, dim3(32 * PH_WARPS), 0, stream, (const T*)x, (TO*)y, p, heads, Dp); \
+    } while (0)
+    if (dtype == RI_DTYPE_F32 && out_dtype == RI_DTYPE_F32) PH_GO(float, float);
+    else if (dtype == RI_DTYPE_F32 && out_dtype == RI_DTYPE_BF16) PH_GO(float, __nv_bfloat16);
+    else if (dtype == RI_DTYPE_BF16 && out_dtype == RI_DTYPE_BF16) PH_GO(__nv_bfloat16, __nv_bfloat16);
+    else RI_FAIL(-1, "pair_heads: dtypes %d and %d", dtype, out_dtype);
 #undef PH_GO
     RI_CHECK_LAUNCH("pair_heads");
     return 0;

@@ -61,7 +61,7 @@ _SIGNATURES = {
     ("norm_gains", "ri_norm_gains"): [_P] * 6 + [_P, _I, _F] + [_P] * 6 + [_I, _I, _F, _I, _P, _I, _I, _P, _P],
     ("dyn_tanh", "ri_dyn_tanh"): [_P] * 7 + [_I, _I, _I, _P, _I, _I, _P],
     ("dyn_tanh", "ri_embed_dyn_tanh"): [_P, _P, _F, _P, _P, _P, _P, _I, _I, _I, _I, _P, _P],
-    ("pair_heads", "ri_pair_heads"): [_P, _P, _F, _F, _F, _I, _I, _I, _I, _I, _I, _P],
+    ("pair_heads", "ri_pair_heads"): [_P, _P, _F, _F, _F, _I, _I, _I, _I, _I, _I, _I, _P],
     ("linear_f32", "ri_linear_f32"): [_P, _P, _P, _I, _I, _I, _P],
     ("sampling", "ri_sample"): [_P, _L, _I, _I, _P, _P, _L, _P, _P, _P, _P, _P, _P, _P, _L, _I, _I, _P, _I, _P],
     ("sampling", "ri_sample_work_bytes"): [_I, _I],
@@ -75,8 +75,8 @@ _SIGNATURES = {
     ("linear_skinny", "ri_linear_skinny_gated_with"): [_P, _P, _P, _I, _I, _I, _I, _F, _F, _P, _P],
     ("linear_stream_tc", "ri_linear_stream_tc"): [_P, _P, _P, _I, _I, _I, _I, _I, _P, _P],
     ("linear_stream_tc", "ri_linear_stream_tc_gate"): [_P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P, _P],
-    ("attention_prefill_tc", "ri_attention_prefill_tc"): [_P] * 8 + [_I] * 9 + [_F, _I, _P, _F, _P, _I, _I, _P, _P],
-    ("attention_prefill", "ri_attention_prefill"): [_P] * 8 + [_I] * 8 + [_F, _I, _P, _I, _F, _P, _I, _I, _P, _P],
+    ("attention_prefill_tc", "ri_attention_prefill_tc"): [_P] * 8 + [_I] * 9 + [_F, _I, _P, _F, _P, _I, _I] + [_I, _I, _I, _F, _F, _F] + [_P, _P],
+    ("attention_prefill", "ri_attention_prefill"): [_P] * 8 + [_I] * 8 + [_F, _I, _P, _I, _F, _P, _I, _I, _I, _P, _P],
 }
 DECODE_CHUNK = 128          # keys per partial result of the decode attention kernel
 MAX_FAST_HEAD_DIM = 256
@@ -886,17 +886,19 @@ def embed_dyn_tanh(ids: torch.Tensor, table: torch.Tensor, scale: float, alpha: 
     return out
 
 
-def pair_heads(x: torch.Tensor, lam: float, eps: float, gain: float, width: int, vdim: int) -> torch.Tensor:
+def pair_heads(x: torch.Tensor, lam: float, eps: float, gain: float, width: int, vdim: int,
+               out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     """The two maps of differential attention put together: x [tokens, 2 H, Dp] holds head h's results a = x[:, 2h] and
     b = x[:, 2h + 1] (``vdim`` true elements); o = a - lam b, then o / sqrt(mean(o^2) + eps) * gain, the mean over ``vdim``
-    elements, all in float32.  Returns [tokens, H, width] (``width`` >= vdim: zeros behind the true elements)."""
+    elements, all in float32.  Returns [tokens, H, width] (``width`` >= vdim: zeros behind the true elements) in x's dtype or in
+    ``out_dtype`` (bfloat16 behind float32)."""
     _need(x, "x")
     tokens, two, Dp = x.shape
     if two % 2 or not 0 < vdim <= min(width, Dp):
         raise KernelError(f"pair_heads: {two} results of {Dp}, {vdim} elements in rows of {width}")
-    out = torch.empty((tokens, two // 2, width), dtype=x.dtype, device=x.device)
+    out = torch.empty((tokens, two // 2, width), dtype=out_dtype or x.dtype, device=x.device)
     _call("pair_heads", "ri_pair_heads", x.data_ptr(), out.data_ptr(), float(lam), float(eps), float(gain), tokens, two // 2, Dp,
-          int(width), int(vdim), _code(x.dtype), _stream())
+          int(width), int(vdim), _code(x.dtype), _code(out.dtype), _stream())
     return out
 
 
@@ -1110,13 +1112,15 @@ def attention_prefill(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tenso
                       seq_slot: torch.Tensor, seq_start: torch.Tensor, seq_len: torch.Tensor, max_new: int,
                       scale: float, window: int, sink: Optional[torch.Tensor] = None, v_dims: int = 0,
                       chunk: int = 0, softcap: float = 0.0, dist_bias: Optional[torch.Tensor] = None,
-                      keep: int = 0) -> torch.Tensor:
+                      keep: int = 0, pair=None, pair_dim: int = 0) -> torch.Tensor:
     """Attention of the step's new tokens (q [tokens, H, Dh], bfloat16, sequences back
     to back as ``seq_start`` says) over the paged cache, which already holds their keys
     and values; ``max_new`` is the most tokens one sequence brings.  ``v_pool`` may be ``k_pool``
     itself (values that are the keys): the mma.sync kernel then reads each tile once; ``v_dims`` > 0
     says that only that many leading elements of the result are wanted (the rest may be zeros).  ``keep`` as for
-    ``attention``."""
+    ``attention``.  ``pair`` as for ``attention_decode`` (``pair_dim``: the elements of one map's queries and keys, which
+    stand side by side in a row): the tcgen05 kernel puts the maps together itself, the mma.sync kernel leaves float32 results
+    for ``pair_heads``; the result is [tokens, H / 2, width]."""
     _need(q, "q", torch.bfloat16)
     tokens, H, Dh = q.shape
     pages, KV, page_size, dh = k_pool.shape
@@ -1131,20 +1135,25 @@ def attention_prefill(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tenso
     _need(seq_slot, "seq_slot", torch.int32, (seqs,))
     _need(seq_start, "seq_start", torch.int32, (seqs + 1,))
     _need(seq_len, "seq_len", torch.int32, (seqs,))
-    out = torch.empty_like(q)
+    lam, eps, gain, width, vdim = pair or (0.0, 0.0, 0.0, 0, 0)
+    if pair is not None and not 0 < 2 * pair_dim <= Dh:
+        raise KernelError(f"attention_prefill: two maps of {pair_dim} elements in rows of {Dh}")
     if Dh in TCGEN05_HEAD_DIMS and not _NO_TCGEN05:
+        out = torch.empty_like(q) if pair is None else torch.empty((tokens, H // 2, width), dtype=q.dtype, device=q.device)
         # head sizes of 64 and 128: the tcgen05 / tensor-memory kernel
         _call("attention_prefill_tc", "ri_attention_prefill_tc", q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(),
               out.data_ptr(), page_table.data_ptr(), seq_slot.data_ptr(), seq_start.data_ptr(), seq_len.data_ptr(),
               q.shape[0], seqs, int(max_new), H, KV, Dh, page_table.shape[1], page_size, pages, float(scale),
-              _mask(window, chunk), _sink(sink, H), _cap(softcap), *_bias(dist_bias, H), int(keep), error_flag(q.device).data_ptr(),
-              _stream(), defines={"RI_HEAD_DIM": Dh})
+              _mask(window, chunk), _sink(sink, H), _cap(softcap), *_bias(dist_bias, H), int(keep), int(width), int(vdim), int(pair_dim),
+              float(lam), float(eps), float(gain), error_flag(q.device).data_ptr(), _stream(), defines={"RI_HEAD_DIM": Dh})
         return out
+    out = torch.empty(q.shape, dtype=q.dtype if pair is None else torch.float32, device=q.device)
     _call("attention_prefill", "ri_attention_prefill", q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(),
           out.data_ptr(), page_table.data_ptr(), seq_slot.data_ptr(), seq_start.data_ptr(), seq_len.data_ptr(),
           seqs, int(max_new), H, KV, Dh, page_table.shape[1], page_size, pages, float(scale), _mask(window, chunk),
-          _sink(sink, H), int(v_dims), _cap(softcap), *_bias(dist_bias, H), int(keep), error_flag(q.device).data_ptr(), _stream(), defines={"RI_HEAD_DIM": Dh})
-    return out
+          _sink(sink, H), int(v_dims), _cap(softcap), *_bias(dist_bias, H), int(keep), 0 if pair is None else 1, error_flag(q.device).data_ptr(),
+          _stream(), defines={"RI_HEAD_DIM": Dh})
+    return out if pair is None else pair_heads(out, *pair, out_dtype=q.dtype)
 
 
 def argmax(logits: torch.Tensor) -> torch.Tensor:

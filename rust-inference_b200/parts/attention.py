@@ -31,8 +31,8 @@ Differential attention (``maps`` 2): a key head's two keys stand side by side in
 one value, so nothing is stored twice.  A query head becomes two query heads of that size, each with its own query in its
 place and zeros in the other's (``ops.qkv_prep``): a zero times a key element adds exactly 0, so its score against the
 whole key is its map's score, and the attention kernels run 2 H heads over the G key heads as they are.  The two maps of a
-head are neighbours; they are put together in float32 by the merge of the decode kernel's partial results, or behind the
-other attention kernels (``ops.pair_heads``): difference, norm over the value's elements, constant factor.
+head are neighbours; they are put together in float32 by the merge of the decode kernel's partial results, by the tcgen05
+prefill kernel at the end of a tile, or behind the other attention kernels (``ops.pair_heads``): difference, norm over the value's elements, constant factor.
 """
 from __future__ import annotations
 
@@ -263,12 +263,12 @@ class Attention(Mixer):
             elif fast:
                 out = ops.attention_prefill(q, cache.k_pool, cache.v_pool, cache.page_table, ctx.seq_slot,
                                             ctx.seq_start, ctx.seq_len, ctx.max_new, self.scale, s.window,
-                                            softcap=self.softcap, dist_bias=self.dist_bias, keep=self.keep)
+                                            softcap=self.softcap, dist_bias=self.dist_bias, keep=self.keep, pair=pair, pair_dim=s.head_dim)
             else:
                 out = ops.attention(q, cache.k_pool, cache.v_pool, cache.page_table, ctx.seq_slot, ctx.seq_start,
                                     ctx.seq_len, ctx.max_new, self.scale, s.window, softcap=self.softcap,
                                     dist_bias=self.dist_bias, keep=self.keep)
-        if pair is not None and not (fast and ctx.decode_only):
+        if pair is not None and not fast:
             with section("attn pairs"):
                 out = ops.pair_heads(out, *pair)
         if self.gated:

@@ -569,8 +569,8 @@ def embed_dyn_tanh(ids, table, scale, alpha, gain, bias):
     return torch.tanh(alpha * (table[ids.long()].float() * scale)) * gain + bias
 
 
-def pair_heads(x, lam, eps, gain, width, vdim):
+def pair_heads(x, lam, eps, gain, width, vdim, out_dtype=None):
     f = x.float()
     o = f[:, 0::2, :vdim] - lam * f[:, 1::2, :vdim]
     o = o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps) * gain
-    return torch.nn.functional.pad(o, (0, width - vdim)).to(x.dtype).contiguous()
+    return torch.nn.functional.pad(o, (0, width - vdim)).to(out_dtype or x.dtype).contiguous()

@@ -267,6 +267,63 @@ def test_pairs_of_maps_are_put_together(T, Hq, Dp, vdim, width, dtype):
     _close(got[:, :, :vdim], P.over_rms(a[:, 0::2] - lam * a[:, 1::2], eps) * gain, dtype, "pairs", tol32=3e-6, tol16=5e-3)
     assert torch.all(got[:, :, vdim:] == 0) and got.shape == (T, Hq, width)
     assert torch.equal(ops.pair_heads(x[T - 1:].contiguous(), lam, eps, gain, width, vdim), got[T - 1:])
+    if dtype == torch.float32:                                      # float32 results of an attention kernel, rounded once
+        got = ops.pair_heads(x, lam, eps, gain, width, vdim, out_dtype=torch.bfloat16)
+        _close(got[:, :, :vdim], P.over_rms(a[:, 0::2] - lam * a[:, 1::2], eps) * gain, torch.bfloat16, "rounded", tol16=5e-3)
+        assert torch.all(got[:, :, vdim:] == 0) and got.dtype == torch.bfloat16
+
+
+@pytest.mark.parametrize("D, dim, vdim, Hq, KV, size, keep", [(128, 64, 128, 8, 2, 200, 4), (64, 32, 64, 2, 1, 0, 0), (128, 20, 120, 4, 4, 70, 40), (64, 30, 33, 6, 1, 33, 1),
+                                                              (96, 48, 96, 4, 1, 40, 6), (128, 60, 17, 2, 2, 129, 128), (48, 17, 34, 20, 1, 64, 3)])
+def test_attention_kernels_put_pairs_together(D, dim, vdim, Hq, KV, size, keep):
+    """Prompts and portions of very different lengths in one step, then one token each: every bfloat16 kernel with the two maps
+    put together in float32, against the plain formulas; the pieces a sequence falls into do not depend on the others."""
+    from rust_inference_b200 import ops
+    rng = np.random.default_rng(D + dim)
+    lengths, news = [300, 1, 45, 129, 460, 77], [300, 1, 2, 129, 130, 33]
+    scale, lam, eps, gain, width = 0.4, 0.7, 1e-3, 0.6, -(-vdim // 16) * 16
+    mask = {"size": size, "keep_first": keep} if size else None
+    pages = sum(-(-n // 32) for n in lengths)
+    kp = torch.zeros((pages, KV, 32, D), dtype=torch.bfloat16, device=DEV)
+    vp = torch.zeros_like(kp)
+    table = torch.full((len(lengths), 16), -1, dtype=torch.int32, device=DEV)
+    ids, at, qs, want = rng.permutation(pages), 0, [], []
+    for b, n in enumerate(lengths):
+        k, v, q = (_t(rng.standard_normal((n, h, d)), torch.bfloat16) for h, d in ((KV, 2 * dim), (KV, vdim), (2 * Hq, dim)))
+        mine = ids[at:at + -(-n // 32)]
+        at += len(mine)
+        table[b, :len(mine)] = _i(mine)
+        for j, page in enumerate(mine):
+            m = min(32, n - 32 * j)
+            kp[page, :, :m, :2 * dim] = k[32 * j:32 * j + m].transpose(0, 1)
+            vp[page, :, :m, :vdim] = v[32 * j:32 * j + m].transpose(0, 1)
+        rows = torch.zeros((n, Hq, 2, D), dtype=torch.bfloat16, device=DEV)
+        rows[:, :, 0, :dim], rows[:, :, 1, dim:2 * dim] = q[:, 0::2], q[:, 1::2]
+        qs.append(rows.view(n, 2 * Hq, D)[n - news[b]:])
+        k64, v64, q64, out = _np(k).reshape(n, KV, 2, dim), _np(v), _np(q).reshape(n, Hq, 2, dim), []
+        for p in range(n - news[b], n):
+            j = P.sees(p, mask)
+            for h in range(Hq):
+                g = h // (Hq // KV)
+                one, two = (P.weighted((k64[j, g, t] @ q64[p, h, t]) * scale, v64[j, g]) for t in (0, 1))
+                out.append(P.over_rms(one - lam * two, eps) * gain)
+        want.append(np.asarray(out).reshape(news[b], Hq, vdim))
+    pair = (lam, eps, gain, width, vdim)
+    start = np.concatenate([[0], np.cumsum(news)])
+    slots = list(range(len(lengths)))
+    got = ops.attention_prefill(torch.cat(qs), kp, vp, table, _i(slots), _i(start), _i(lengths), max(news), scale, size, keep=keep,
+                                pair=pair, pair_dim=dim)
+    assert got.shape == (sum(news), Hq, width) and torch.all(got[:, :, vdim:] == 0)
+    _close(got[:, :, :vdim], np.concatenate(want), torch.bfloat16, "prompts together", tol16=3e-2)
+    for b in slots:
+        alone = ops.attention_prefill(qs[b].contiguous(), kp, vp, table, _i([b]), _i([0, news[b]]), _i([lengths[b]]), news[b], scale, size,
+                                      keep=keep, pair=pair, pair_dim=dim)
+        assert torch.equal(alone, got[start[b]:start[b + 1]]), f"sequence {b} alone"
+    last = torch.cat([q[-1:] for q in qs])
+    got = ops.attention_decode(last, kp, vp, table, _i(slots), _i(lengths), scale, size, 1024, keep=keep, pair=pair)
+    assert torch.all(got[:, :, vdim:] == 0)
+    _close(got[:, :, :vdim], np.stack([w[-1] for w in want]), torch.bfloat16, "one token each", tol16=3e-2)
+    _no_error()
 
 
 def _mixer(spec, dtype, w):
