@@ -376,8 +376,8 @@ def zavevik_config(z) -> dict:
 
 
 def gotulorn_config(z) -> dict:
-    """Layers in turns of three: differential attention (half as many heads as the width has parts of 128, each with two maps
-    of 64 and a value of 128, four heads per key/value head, a window of 2,048 beside 4 kept tokens), latent attention (per
+    """Layers in turns of three: differential attention (heads of two maps of 64 and a value of 128, four heads per
+    key/value head, a window of 2,048 beside 4 kept tokens), latent attention (per
     head 128 plain and 64 rotated elements, a latent of 192), differential attention over the keys and values of the first.
     Feed-forwards take turns: dense, and routed (16 experts of an eighth of the dense width, 4 per token)."""
     D, H = z["width"], z["heads"]
