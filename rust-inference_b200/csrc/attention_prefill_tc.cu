@@ -37,7 +37,7 @@
 //   k_empty[s], v_empty[s] (both issuing lanes: tcgen05.commit, or a plain arrival for a block left out)  stage s is free
 //   q_full[t]  (TMA)                the item's queries of tile t have landed
 //   q_empty[t] (tcgen05.commit)     the item's last product Q_t K^T is done: the next item's queries may come
-//   o_free[t]  (4 arrivals)         the tile's threads hold the item's output: the next item's first product may overwrite O_t
+//   o_free[t]  (4 arrivals; PAIR: 8) the tile's (PAIR: all) threads hold the item's output: the next item's first product may overwrite O_t
 // Every barrier belongs to one buffer; a barrier waited on by parity is never two phases ahead of a
 // waiter, because its next phase needs something that waiter does after the wait.  Every wait is
 // bounded by time and ends in an error code (5), not a hang: the thread that gave up says so in shared memory,
@@ -56,9 +56,10 @@
 // Differential attention (PAIR, a variant of its own; pair_heads.cuh has the formula): an item is ONE query tile of 128 tokens
 // and one pair of heads, the two maps over the same values; tile 0 is the first map, tile 1 the second.  Both see the same
 // blocks of keys.  A map's query is zero outside its own half of the row, so its product with the keys takes only the k steps
-// of that half.  At the end of an item tile 1's threads hand the reciprocals of their rows' sums over in shared memory, and tile
-// 0's threads read both outputs from tensor memory (a thread reaches its row's lane in the columns of either tile), take the
-// difference, norm it and store it: nothing is rounded before that.
+// of that half.  At the end of an item the two threads of a row (one per tile) exchange the reciprocals of their sums in shared
+// memory; each reads half of the columns of BOTH outputs from tensor memory (a thread reaches its row's lane in the columns of
+// either tile) and takes the difference, they exchange their halves' sums of squares, and each norms and stores its half:
+// nothing is rounded before that.
 //
 // Compile with -DRI_HEAD_DIM=64 or 128.  Page size is 32.
 // Formula: thanhauco/rust-inference src/attention.rs:4-8, 111-150.
@@ -278,9 +279,10 @@ struct TcTail {
     unsigned long long q_full[2], q_empty[2], o_free[2];
     unsigned tmem_base;
     volatile int dead;
-    float pair_inv[TC_BM];              // 1 / (sum of the row's weights) of tile 1, for tile 0's threads
+    float pair_inv[2][TC_BM];           // 1 / (sum of the row's weights) of either tile
+    float pair_ss[2][TC_BM];            // sums of squares of either half of the row's difference
 };
-#define TC_SMEM_BYTES (TC_OFF_TAIL + 448 + TC_BM * 4)
+#define TC_SMEM_BYTES (TC_OFF_TAIL + 448 + 4 * TC_BM * 4)
 #define TC_TMEM_COLS 512
 #define TC_S_COL(t, b) (((t) * 2 + (b)) * TC_BN)       // two S buffers per tile
 #define TC_O_COL(t) (4 * TC_BN + (t) * 128)
@@ -383,7 +385,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;\n" ::"r"(smem_u32(&tail.pv_done[i][1])));
             asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;\n" ::"r"(smem_u32(&tail.q_full[i])));
             asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;\n" ::"r"(smem_u32(&tail.q_empty[i])));
-            asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;\n" ::"r"(smem_u32(&tail.o_free[i])), "r"(TC_BM / 32));
+            asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;\n" ::"r"(smem_u32(&tail.o_free[i])), "r"((PAIR ? 2 : 1) * TC_BM / 32));
 #pragma unroll
             for (int b2 = 0; b2 < 2; b2++) {
                 asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;\n" ::"r"(smem_u32(&tail.p_ready[i][b2])), "r"(TC_BM / 32));
@@ -754,54 +756,46 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             if (work.sink && m != -FLT_MAX) l += ex2_approx(work.sink[it.h] * 1.4426950408889634f - m);
             const float inv = 1.0f / l;
             if (PAIR) {
-                // both tiles' threads have the item's outputs in tensor memory behind this barrier
-                if (t == 1) tail.pair_inv[row] = inv;
+                constexpr int HALF = TC_DH / 2;                       // columns of this thread: t HALF .. t HALF + HALF - 1
+                const PairOut& pr = work.pair;
+                tail.pair_inv[t][row] = inv;
                 tc_fence_before();
                 asm volatile("bar.sync 1, %0;\n" ::"n"(32 * 4 * TC_TILES) : "memory");
-                tc_fence_after();
-                if (t == 0) {
-                    const PairOut& pr = work.pair;
-                    const float inv1 = pr.lam * tail.pair_inv[row];
-                    float ss = 0.0f;
+                tc_fence_after();                                     // both tiles' outputs stand in tensor memory
+                const float inv0 = tail.pair_inv[0][row], inv1 = pr.lam * tail.pair_inv[1][row];
+                const int col0 = t * HALF;
+                float o[HALF];
+                float ss = 0.0f;
 #pragma unroll
-                    for (int cc = 0; cc < TC_DH / 32; cc++) {
-                        float a[32], b[32];
-                        tmem_ld32(tmem_row + TC_O_COL(0) + cc * 32, a);
-                        tmem_ld32(tmem_row + TC_O_COL(1) + cc * 32, b);
+                for (int cc = 0; cc < HALF / 32; cc++) {
+                    unsigned a[32], b[32];
+                    tmem_ld32_start(tmem_row + TC_O_COL(0) + col0 + cc * 32, a);
+                    tmem_ld32_start(tmem_row + TC_O_COL(1) + col0 + cc * 32, b);
+                    tmem_ld_wait();
 #pragma unroll
-                        for (int i = 0; i < 32; i++) {
-                            const float o = a[i] * inv - b[i] * inv1;
-                            ss += cc * 32 + i < pr.vdim ? o * o : 0.0f;
-                        }
+                    for (int i = 0; i < 32; i++) {
+                        const float d = __uint_as_float(a[i]) * inv0 - __uint_as_float(b[i]) * inv1;
+                        o[cc * 32 + i] = col0 + cc * 32 + i < pr.vdim ? d : 0.0f;
+                        ss += o[cc * 32 + i] * o[cc * 32 + i];
                     }
-                    const float f = pr.gain / sqrtf(ss / (float)pr.vdim + pr.eps);
-                    bf16* dst = out + ((size_t)(it.t_first + (mine ? row : 0)) * (H / 2) + it.h / 2) * pr.width;
+                }
+                // my columns of both outputs are in my registers: the next item's first products may overwrite them
+                tc_fence_before();
+                __syncwarp();
+                if (lane == 0) {
+                    asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(smem_u32(&tail.o_free[0])) : "memory");
+                    asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(smem_u32(&tail.o_free[1])) : "memory");
+                }
+                tail.pair_ss[t][row] = ss;
+                asm volatile("bar.sync 1, %0;\n" ::"n"(32 * 4 * TC_TILES) : "memory");
+                const float f = pr.gain / sqrtf((tail.pair_ss[0][row] + tail.pair_ss[1][row]) / (float)pr.vdim + pr.eps);
+                if (mine) {
+                    bf16* dst = out + ((size_t)(it.t_first + row) * (H / 2) + it.h / 2) * pr.width + col0;
 #pragma unroll
-                    for (int cc = 0; cc < TC_DH / 32; cc++) {
-                        float a[32], b[32];
-                        tmem_ld32(tmem_row + TC_O_COL(0) + cc * 32, a);
-                        tmem_ld32(tmem_row + TC_O_COL(1) + cc * 32, b);
-                        if (mine) {
-#pragma unroll
-                            for (int i = 0; i < 32; i += 8) {
-                                if (cc * 32 + i >= pr.width) continue;
-                                float y[8];
-#pragma unroll
-                                for (int e = 0; e < 8; e++)
-                                    y[e] = cc * 32 + i + e < pr.vdim ? (a[i + e] * inv - b[i + e] * inv1) * f : 0.0f;
-                                *(uint4*)(dst + cc * 32 + i) = make_uint4(pack_bf16(y[0], y[1]), pack_bf16(y[2], y[3]),
-                                                                          pack_bf16(y[4], y[5]), pack_bf16(y[6], y[7]));
-                            }
-                        }
-                    }
-                    // both outputs have been read: the next item's first products may overwrite them (tile 1's threads write
-                    // pair_inv again only behind the next item's products)
-                    tc_fence_before();
-                    __syncwarp();
-                    if (lane == 0) {
-                        asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(smem_u32(&tail.o_free[0])) : "memory");
-                        asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(smem_u32(&tail.o_free[1])) : "memory");
-                    }
+                    for (int i = 0; i < HALF; i += 8)
+                        if (col0 + i < pr.width)
+                            *(uint4*)(dst + i) = make_uint4(pack_bf16(o[i] * f, o[i + 1] * f), pack_bf16(o[i + 2] * f, o[i + 3] * f),
+                                                            pack_bf16(o[i + 4] * f, o[i + 5] * f), pack_bf16(o[i + 6] * f, o[i + 7] * f));
                 }
                 c += my_blocks;
                 kv_base += it.n_blocks;
