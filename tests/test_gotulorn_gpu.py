@@ -132,9 +132,9 @@ def _plain_masked(q, k, v, scale, mask, positions):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("D, Hq, KV, size, keep", [(32, 4, 2, 40, 6), (80, 4, 4, 1, 1), (64, 4, 2, 70, 33), (128, 4, 1, 64, 64),
+@pytest.mark.parametrize("D, Hq, KV, size, keep", [(32, 4, 2, 43, 7), (80, 4, 4, 1, 1), (64, 4, 2, 70, 33), (128, 4, 1, 64, 64),
                                                    (64, 20, 1, 31, 3), (48, 3, 1, 200, 129), (128, 2, 2, 129, 0), (64, 2, 1, 33, 300),
-                                                   (22, 2, 1, 50, 32), (144, 6, 2, 40, 6), (128, 8, 2, 300, 1)])
+                                                   (22, 2, 1, 50, 32), (176, 6, 2, 45, 5), (128, 8, 2, 300, 1)])
 def test_attention_with_kept_first_tokens(D, Hq, KV, size, keep, dtype):
     """A query that sees one of the loud keys hears nothing else: they stand further apart than the window is long, the first one
     right behind the kept tokens, and the last kept token is loud where none of them is in sight, so that one key too many or
@@ -274,7 +274,7 @@ def test_pairs_of_maps_are_put_together(T, Hq, Dp, vdim, width, dtype):
 
 
 @pytest.mark.parametrize("D, dim, vdim, Hq, KV, size, keep", [(128, 64, 128, 8, 2, 200, 4), (64, 32, 64, 2, 1, 0, 0), (128, 20, 120, 4, 4, 70, 40), (64, 30, 33, 6, 1, 33, 1),
-                                                              (96, 48, 96, 4, 1, 40, 6), (128, 60, 17, 2, 2, 129, 128), (48, 17, 34, 20, 1, 64, 3)])
+                                                              (96, 40, 88, 6, 2, 45, 7), (128, 60, 17, 2, 2, 129, 128), (48, 17, 34, 20, 1, 64, 3)])
 def test_attention_kernels_put_pairs_together(D, dim, vdim, Hq, KV, size, keep):
     """Prompts and portions of very different lengths in one step, then one token each: every bfloat16 kernel with the two maps
     put together in float32, against the plain formulas; the pieces a sequence falls into do not depend on the others."""
@@ -557,7 +557,7 @@ def test_a_far_key_among_hundreds_is_found(tmp_path, kind, far, dtype):
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("borrowed", [False, True])
-@pytest.mark.parametrize("size, keep", [(40, 6), (33, 32), (64, 33), (31, 1), (97, 0)])
+@pytest.mark.parametrize("size, keep", [(44, 7), (33, 32), (64, 33), (31, 1), (97, 0)])
 def test_keys_at_the_edges_of_window_and_kept_tokens(tmp_path, size, keep, borrowed, dtype):
     """Some positions look for the key just inside the window, some for the one just outside, some for the first and the last
     kept token and the one behind it.  A mask that is one token off in any way would show."""
